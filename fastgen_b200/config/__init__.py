@@ -17,6 +17,7 @@ from . import sinorax as _sinorax  # registers Sinorax
 from . import zeladra as _zeladra  # registers Zeladra
 from . import tanupel as _tanupel  # registers Tanupel
 from . import palulorn as _palulorn  # registers Palulorn
+from . import kuvusun as _kuvusun  # registers Kuvusun
 
 __all__ = [
     "ConfigError",

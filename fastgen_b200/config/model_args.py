@@ -93,6 +93,8 @@ class ModelArgs:
     #: how token ids become the first residual stream (``None``: a plain table named
     #: ``embedding_name``); its ``"table"`` tensor is what a tied output projection uses
     embedder: Optional[PartSpec] = None
+    #: a norm that the embedder's output passes on its way into the residual stream (``None``: none)
+    embed_norm: Optional[PartSpec] = None
     #: logits are multiplied by ``logit_scale`` and then, with a cap, squashed to
     #: ``cap * tanh(logits / cap)``
     logit_scale: float = 1.0
@@ -112,6 +114,8 @@ class ModelArgs:
 
     def __post_init__(self) -> None:
         n = len(self.layers)
+        if self.embed_norm is not None and self.streams is not None:
+            raise ConfigError("the embedder's output is normed into one residual stream, not into several")
         if any(e.mix_input for e in self.schedule):
             if self.pass_input_name is None:
                 raise ConfigError("a schedule entry mixes the embedder's output in, but the model names no tensor for it")

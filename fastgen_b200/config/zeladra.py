@@ -104,7 +104,7 @@ def _latent_attention(dim: int, eps: float, m: Mapping[str, Any], prefix: str, w
         eps=eps,
         position=_rope(m["rot"], rot_dim, where),
         own_cache=own,
-        gate=True,
+        gate="head",
     )
     names = {"w_dq": "dq", "dq_norm": "dq.norm", "w_uq": "uq", "w_uk": "uk", "w_uv": "uv", "w_g": "g", "wo": "o"}
     if own:

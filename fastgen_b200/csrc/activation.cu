@@ -129,9 +129,40 @@ head_gate_bf16x8_kernel(__nv_bfloat16* x, long x_stride, const __nv_bfloat16* __
   *p = raw;
 }
 
+// One gate a column (head_dim 1), both sides in 16-byte pieces of bfloat16.
+__global__ void __launch_bounds__(256)
+column_gate_bf16x8_kernel(__nv_bfloat16* x, long x_stride, const __nv_bfloat16* gate, long gate_stride,
+                          const int* __restrict__ req, int n_tokens, int width) {
+  const int pieces = width / 8;  // a row's
+  const long idx = (long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (idx >= (long)n_tokens * pieces) return;
+  const int t = (int)(idx / pieces), piece = (int)(idx - (long)t * pieces);
+  if (req != nullptr && req[t] < 0) return;
+  const uint4 graw = *reinterpret_cast<const uint4*>(gate + (size_t)t * gate_stride + piece * 8);
+  uint4* p = reinterpret_cast<uint4*>(x + (size_t)t * x_stride + piece * 8);
+  uint4 raw = *p;
+  __nv_bfloat162* h2 = reinterpret_cast<__nv_bfloat162*>(&raw);
+  const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&graw);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const float2 v = __bfloat1622float2(h2[i]), g = __bfloat1622float2(g2[i]);
+    // the special-function unit's exponential and reciprocal, as in silu_gate.cu: far below the rounding
+    h2[i] = __floats2bfloat162_rn(__fdividef(v.x, 1.f + __expf(-g.x)), __fdividef(v.y, 1.f + __expf(-g.y)));
+  }
+  *p = raw;
+}
+
 extern "C" int fg_head_gate(void* x, long x_stride, const void* gate, long gate_stride, int dtype, const int* req,
                             int n_tokens, int heads, int head_dim, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
+  if (dtype == FG_BF16 && head_dim == 1 && heads % 8 == 0 && x_stride % 8 == 0 && gate_stride % 8 == 0 &&
+      ((uintptr_t)x & 15) == 0 && ((uintptr_t)gate & 15) == 0) {
+    const long n = (long)n_tokens * heads / 8;
+    column_gate_bf16x8_kernel<<<(unsigned)((n + 255) / 256), 256, 0, stream>>>(
+        (__nv_bfloat16*)x, x_stride, (const __nv_bfloat16*)gate, gate_stride, req, n_tokens, heads);
+    FG_CHECK_LAUNCH("fg_head_gate");
+    return 0;
+  }
   if (dtype == FG_BF16 && head_dim % 8 == 0 && x_stride % 8 == 0 && ((uintptr_t)x & 15) == 0) {
     const long n = (long)n_tokens * heads * head_dim / 8;
     head_gate_bf16x8_kernel<<<(unsigned)((n + 255) / 256), 256, 0, stream>>>(

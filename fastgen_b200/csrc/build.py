@@ -40,6 +40,7 @@ CORE_SOURCES = [
     "embedding.cu",
     "rmsnorm.cu",
     "rmsnorm_sum.cu",
+    "part_norm.cu",
     "dyt.cu",
     "stream_norm.cu",
     "mamba2.cu",

@@ -1,7 +1,7 @@
 // Feed-forward with routed experts: every token goes through `top` of `n_experts` small gated
 // feed-forwards and their outputs are summed with the router's weights.
 //
-//   fg_moe_logits  the router's logits x W^T in float32 (W float32, x of either type): a warp a token.
+//   fg_moe_logits  the router's logits x W^T + b in float32 (W, b float32, x of either type): a block a token.
 //   fg_moe_route   scores s = softmax(logits) (float32); the experts with the largest s + correction
 //                  are chosen; their weights are their s, as they are (or divided by their sum).
 //   fg_moe_plan    sorts the (token, choice) pairs by expert (stable: ascending pair index within an
@@ -13,11 +13,12 @@
 //                  with two weight stacks the result is silu(x W1^T) * (x W3^T).  This is the product of
 //                  the float32 mode and of sizes the tensor-core kernel does not take.
 //   fg_moe_gemm_mma the same product in bfloat16 on the tensor cores.
-//   fg_moe_combine ff[t, :] = sum_k weight[t, k] * y[row of (t, k), :], ascending k.
+//   fg_moe_combine ff[t, :] = sum_k weight[t, k] * y[row of (t, k), :], ascending k, and with a shared expert
+//                  that has a gate + sigmoid(gate[t]) * shared[t, :].
 #include "common.cuh"
 
 // ---- the router's logits ---------------------------------------------------------------------
-// logits[t, e] = sum_k x[t, k] w[e, k] in float32: a block of four warps a token, eight experts at a
+// logits[t, e] = sum_k x[t, k] w[e, k] (+ bias[e]) in float32: a block of four warps a token, eight experts at a
 // time.  A thread sums runs of eight consecutive k (read as 16-byte words, all of an expert group's
 // loads in flight before the first sum: the router's matrix comes from memory at every step and a
 // chain of dependent loads would be all latency) in ascending order; the threads' sums meet in a fixed
@@ -47,8 +48,8 @@ __device__ __forceinline__ void load8<__nv_bfloat16>(const __nv_bfloat16* p, flo
 
 template <typename T, bool VEC>
 __global__ void __launch_bounds__(LOGITS_THREADS)
-moe_logits_kernel(const T* x, long ldx, const float* __restrict__ w, long ldw, float* __restrict__ logits,
-                  const int* __restrict__ req, int n_experts, int K) {
+moe_logits_kernel(const T* x, long ldx, const float* __restrict__ w, long ldw, const float* __restrict__ bias,
+                  float* __restrict__ logits, const int* __restrict__ req, int n_experts, int K) {
   __shared__ float part[LOGITS_THREADS / 32][LOGITS_GROUP];
   const int t = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   if (req != nullptr && req[t] < 0) return;
@@ -90,21 +91,22 @@ moe_logits_kernel(const T* x, long ldx, const float* __restrict__ w, long ldw, f
       float total = part[0][tid];
 #pragma unroll
       for (int i = 1; i < LOGITS_THREADS / 32; ++i) total += part[i][tid];
-      logits[(size_t)t * n_experts + e0 + tid] = total;
+      logits[(size_t)t * n_experts + e0 + tid] = bias != nullptr ? total + bias[e0 + tid] : total;
     }
     __syncthreads();
   }
 }
 
-extern "C" int fg_moe_logits(const void* x, int dtype, long ldx, const float* w, long ldw, float* logits,
-                             const int* req, int n_tokens, int n_experts, int K, cudaStream_t stream) {
+extern "C" int fg_moe_logits(const void* x, int dtype, long ldx, const float* w, long ldw, const float* bias,
+                             float* logits, const int* req, int n_tokens, int n_experts, int K, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   FG_CHECK_ARG(n_experts >= 1 && K >= 1, "fg_moe_logits: %d experts over %d inputs", n_experts, K);
   FG_CHECK_ARG(dtype == FG_F32 || dtype == FG_BF16, "fg_moe_logits: bad dtype %d", dtype);
   const long x_words = dtype == FG_F32 ? 4 : 8;  // elements of 16 bytes
   const bool vec = K % 8 == 0 && ((uintptr_t)x & 15) == 0 && ldx % x_words == 0 && ((uintptr_t)w & 15) == 0 && ldw % 4 == 0;
 #define LAUNCH(T, VEC)                                                                                             \
-  moe_logits_kernel<T, VEC><<<n_tokens, LOGITS_THREADS, 0, stream>>>((const T*)x, ldx, w, ldw, logits, req, n_experts, K)
+  moe_logits_kernel<T, VEC><<<n_tokens, LOGITS_THREADS, 0, stream>>>((const T*)x, ldx, w, ldw, bias, logits, req, \
+                                                                     n_experts, K)
   if (dtype == FG_F32) {
     if (vec) LAUNCH(float, true); else LAUNCH(float, false);
   } else {
@@ -118,7 +120,7 @@ extern "C" int fg_moe_logits(const void* x, int dtype, long ldx, const float* w,
 constexpr int ROUTE_MAX_PER_LANE = 8;  // up to 256 experts
 
 __global__ void __launch_bounds__(128)
-moe_route_kernel(const float* logits, const float* __restrict__ correction, int* __restrict__ ids,
+moe_route_kernel(const float* logits, long ldl, const float* __restrict__ correction, int* __restrict__ ids,
                  float* __restrict__ weights, const int* __restrict__ req, int n_tokens, int n_experts, int top,
                  int renormalize) {
   const int t = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
@@ -135,7 +137,7 @@ moe_route_kernel(const float* logits, const float* __restrict__ correction, int*
 #pragma unroll
   for (int i = 0; i < ROUTE_MAX_PER_LANE; ++i) {
     const int e = lane + 32 * i;
-    z[i] = e < n_experts ? logits[(size_t)t * n_experts + e] : -INFINITY;
+    z[i] = e < n_experts ? logits[(size_t)t * ldl + e] : -INFINITY;
     m = fmaxf(m, z[i]);
   }
   m = warp_max(m);
@@ -150,7 +152,8 @@ moe_route_kernel(const float* logits, const float* __restrict__ correction, int*
   for (int i = 0; i < ROUTE_MAX_PER_LANE; ++i) {
     const int e = lane + 32 * i;
     s[i] = s[i] / sum;
-    c[i] = e < n_experts ? s[i] + (correction ? correction[e] : 0.f) : -INFINITY;
+    // (without a correction the logits themselves rank the experts: scores may round to equal)
+    c[i] = e < n_experts ? (correction ? s[i] + correction[e] : z[i]) : -INFINITY;
   }
   for (int k = 0; k < top; ++k) {
     // the largest choice score left; equal scores go to the lower index
@@ -194,14 +197,14 @@ moe_route_kernel(const float* logits, const float* __restrict__ correction, int*
   }
 }
 
-extern "C" int fg_moe_route(const float* logits, const float* correction, int* ids, float* weights, const int* req,
+extern "C" int fg_moe_route(const float* logits, long ldl, const float* correction, int* ids, float* weights, const int* req,
                             int n_tokens, int n_experts, int top, int renormalize, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   FG_CHECK_ARG(n_experts >= 1 && n_experts <= 32 * ROUTE_MAX_PER_LANE, "fg_moe_route: %d experts (1 to %d)",
                n_experts, 32 * ROUTE_MAX_PER_LANE);
   FG_CHECK_ARG(top >= 1 && top <= n_experts, "fg_moe_route: %d of %d experts", top, n_experts);
-  moe_route_kernel<<<(n_tokens + 3) / 4, 128, 0, stream>>>(logits, correction, ids, weights, req, n_tokens, n_experts,
-                                                           top, renormalize);
+  moe_route_kernel<<<(n_tokens + 3) / 4, 128, 0, stream>>>(logits, ldl, correction, ids, weights, req, n_tokens,
+                                                           n_experts, top, renormalize);
   FG_CHECK_LAUNCH("fg_moe_route");
   return 0;
 }
@@ -216,7 +219,7 @@ extern "C" int fg_moe_route(const float* logits, const float* correction, int* i
 constexpr int ROUTE_WARPS = 4;
 
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
-moe_route_groups_kernel(const float* logits, const float* __restrict__ correction, int* __restrict__ ids,
+moe_route_groups_kernel(const float* logits, long ldl, const float* __restrict__ correction, int* __restrict__ ids,
                         float* __restrict__ weights, const int* __restrict__ req, int n_tokens, int n_experts, int top,
                         int kind, int n_groups, int keep_groups, int group_top, int renormalize, float renorm_eps,
                         float weight_scale) {
@@ -238,7 +241,7 @@ moe_route_groups_kernel(const float* logits, const float* __restrict__ correctio
 #pragma unroll
     for (int i = 0; i < ROUTE_MAX_PER_LANE; ++i) {
       const int e = lane + 32 * i;
-      s[i] = e < n_experts ? logits[(size_t)t * n_experts + e] : -INFINITY;
+      s[i] = e < n_experts ? logits[(size_t)t * ldl + e] : -INFINITY;
       m = fmaxf(m, s[i]);
     }
     m = warp_max(m);
@@ -255,7 +258,7 @@ moe_route_groups_kernel(const float* logits, const float* __restrict__ correctio
 #pragma unroll
     for (int i = 0; i < ROUTE_MAX_PER_LANE; ++i) {
       const int e = lane + 32 * i;
-      s[i] = e < n_experts ? 1.f / (1.f + expf(-logits[(size_t)t * n_experts + e])) : 0.f;
+      s[i] = e < n_experts ? 1.f / (1.f + expf(-logits[(size_t)t * ldl + e])) : 0.f;
     }
   }
 #pragma unroll
@@ -347,7 +350,7 @@ moe_route_groups_kernel(const float* logits, const float* __restrict__ correctio
     }
 }
 
-extern "C" int fg_moe_route_groups(const float* logits, const float* correction, int* ids, float* weights,
+extern "C" int fg_moe_route_groups(const float* logits, long ldl, const float* correction, int* ids, float* weights,
                                    const int* req, int n_tokens, int n_experts, int top, int kind, int n_groups,
                                    int keep_groups, int group_top, int renormalize, float renorm_eps,
                                    float weight_scale, cudaStream_t stream) {
@@ -363,7 +366,7 @@ extern "C" int fg_moe_route_groups(const float* logits, const float* correction,
                  keep_groups, top);
   }
   moe_route_groups_kernel<<<(n_tokens + ROUTE_WARPS - 1) / ROUTE_WARPS, ROUTE_WARPS * 32, 0, stream>>>(
-      logits, correction, ids, weights, req, n_tokens, n_experts, top, kind, n_groups, keep_groups, group_top,
+      logits, ldl, correction, ids, weights, req, n_tokens, n_experts, top, kind, n_groups, keep_groups, group_top,
       renormalize, renorm_eps, weight_scale);
   FG_CHECK_LAUNCH("fg_moe_route_groups");
   return 0;
@@ -753,27 +756,31 @@ extern "C" int fg_moe_gemm_mma(const void* x, long ldx, const void* w1, const vo
 // ---- the weighted sum of a token's experts ----------------------------------------------------------
 template <typename T>
 __global__ void __launch_bounds__(256)
-moe_combine_kernel(const T* y, long ldy, const float* weights, const int* pair_row, T* __restrict__ out, long ldo,
-                   int dim, int top) {
+moe_combine_kernel(const T* y, long ldy, const float* weights, const int* pair_row, const T* shared, long lds,
+                   const float* gate, long ldg, T* __restrict__ out, long ldo, int dim, int top) {
   const int t = blockIdx.x;
+  const float g = gate != nullptr ? 1.f / (1.f + expf(-gate[(size_t)t * ldg])) : 1.f;
   for (int c = threadIdx.x; c < dim; c += blockDim.x) {
     float acc = 0.f;
     for (int k = 0; k < top; ++k) {
       const int r = pair_row[(size_t)t * top + k];
       if (r >= 0) acc = fmaf(weights[(size_t)t * top + k], to_f32<T>(y[(size_t)r * ldy + c]), acc);
     }
+    if (shared != nullptr) acc = fmaf(g, to_f32<T>(shared[(size_t)t * lds + c]), acc);
     out[(size_t)t * ldo + c] = from_f32<T>(acc);
   }
 }
 
-extern "C" int fg_moe_combine(const void* y, long ldy, const float* weights, const int* pair_row, void* out, long ldo,
-                              int dtype, int n_tokens, int dim, int top, cudaStream_t stream) {
+// shared: [n_tokens, dim] or null (added, times sigmoid(gate[t * ldg]) with a gate)
+extern "C" int fg_moe_combine(const void* y, long ldy, const float* weights, const int* pair_row, const void* shared,
+                              long lds, const float* gate, long ldg, void* out, long ldo, int dtype, int n_tokens, int dim, int top, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   if (dtype == FG_F32)
-    moe_combine_kernel<float><<<n_tokens, 256, 0, stream>>>((const float*)y, ldy, weights, pair_row, (float*)out, ldo,
-                                                            dim, top);
+    moe_combine_kernel<float><<<n_tokens, 256, 0, stream>>>((const float*)y, ldy, weights, pair_row, (const float*)shared, lds,
+                                                            gate, ldg, (float*)out, ldo, dim, top);
   else if (dtype == FG_BF16)
     moe_combine_kernel<__nv_bfloat16><<<n_tokens, 256, 0, stream>>>((const __nv_bfloat16*)y, ldy, weights, pair_row,
+                                                                    (const __nv_bfloat16*)shared, lds, gate, ldg,
                                                                     (__nv_bfloat16*)out, ldo, dim, top);
   else
     FG_CHECK_ARG(false, "fg_moe_combine: bad dtype %d", dtype);

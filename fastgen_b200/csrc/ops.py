@@ -67,6 +67,7 @@ _CORE_SIGNATURES = {
                          _P, _I, _P],
     "fg_qk_rstd": [_P, _L, _I, _I, _P, _L, _I, _I, _I, _P, _F, _P, _I, _P],
     "fg_rmsnorm_sum": [_P, _P, _P, _I, _I, _P, _P, _I, _I, _P, _I, _P, _I, _I, _F, _P],
+    "fg_part_norm": [_P, _I, _P, _I, _P, _P, _P, _I, _P, _I, _I, _I, _F, _P],
     "fg_gemm_f32_nt_from": [_P, _I, _I, _P, _I, _P, _I, _I, _I, _I, _P],
     "fg_gemm_f32_nt": [_P, _I, _P, _I, _P, _I, _I, _I, _I, _P, _P],
     "fg_gemm_skinny_bf16": [_P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _P, _I, _P],
@@ -190,14 +191,14 @@ _DELTA_SIGNATURES = {
     "fg_head_norm_gate": [_P, _L, _P, _L, _I, _P, _P, _L, _P, _I, _I, _I, _F, _P],
 }
 _MOE_SIGNATURES = {
-    "fg_moe_logits": [_P, _I, _L, _P, _L, _P, _P, _I, _I, _I, _P],
-    "fg_moe_route": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _P],
-    "fg_moe_route_groups": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _P],
+    "fg_moe_logits": [_P, _I, _L, _P, _L, _P, _P, _P, _I, _I, _I, _P],
+    "fg_moe_route": [_P, _L, _P, _P, _P, _P, _I, _I, _I, _I, _P],
+    "fg_moe_route_groups": [_P, _L, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _P],
     "fg_moe_plan": [_P, _I, _I, _I, _P, _P, _P, _P, _P, _P, _I, _P, _P],
     "fg_moe_gather": [_P, _L, _P, _L, _I, _P, _P, _I, _I, _I, _I, _P],
     "fg_moe_gemm": [_P, _L, _P, _P, _L, _P, _L, _I, _I, _I, _P, _I, _P, _P, _P, _P, _I, _P],
     "fg_moe_gemm_mma": [_P, _L, _P, _P, _L, _P, _L, _I, _I, _P, _I, _P, _P, _P, _P, _I, _P],
-    "fg_moe_combine": [_P, _L, _P, _P, _P, _L, _I, _I, _I, _I, _P],
+    "fg_moe_combine": [_P, _L, _P, _P, _P, _L, _P, _L, _P, _L, _I, _I, _I, _I, _P],
 }
 _RECUR_SIGNATURES = {
     "fg_mlstm_scan": [_P, _P, _F, _P, _L, _P, _L, _P, _L, _I, _P, _P, _L, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _F,
@@ -505,9 +506,11 @@ class Ops:
         """Causal softmax attention of ``n_heads`` query heads on the one cached entry per token:
         score ``(qa_h . c + qt_h . k_t) * scale``, output the weighted sum of the latents ``c``, times
         ``sigmoid(gate[t, h])`` when a gate is given.  ``qa`` [heads, T, rank] (folded queries),
-        ``qt`` [T, heads, rot_dim] (a strided view), ``out`` [heads, T, rank], ``gate`` [T, heads]
+        ``qt`` [T, heads, rot_dim] (a strided view; ``rot_dim`` may be 0), ``out`` [heads, T, rank], ``gate`` [T, heads]
         (a strided view) or ``None``."""
         pages = memory.k_pages
+        if rot_dim == 0:
+            qt = qa.permute(1, 0, 2)  # never read: a valid address with even strides
         assert qa.stride(2) == 1 and qt.stride(2) == 1 and out.stride(2) == 1 and pages.is_contiguous()
         assert gate is None or gate.stride(1) == 1
         even = all(v % 2 == 0 for v in (*qa.stride()[:2], *qt.stride()[:2], *out.stride()[:2], qt.storage_offset()))
@@ -646,6 +649,28 @@ class Ops:
             _code(out.dtype) if out is not None else 0, _ptr(rows), n, dim, float(eps), _stream()))
         return out
 
+    def part_norm(self, parts: int, eps: float, h=None, delta=None, delta_weight=None, weight=None, out=None, rows=None,
+                  fresh: bool = False):
+        """RMS norms in ``parts`` equal consecutive parts of a row (float32 arithmetic):
+        ``h += norm(delta) * delta_weight`` (``fresh``: ``h`` becomes it), stored back, then ``out = h``, or
+        ``out = norm(h) * weight`` with a ``weight``.  ``h`` float32 [T, dim]; without ``h``, ``out`` receives
+        the summand's norm; without ``delta``, ``h`` stays as it is.  With ``rows`` (int32 indices) only
+        those rows are computed, into ``out``, and ``h`` is left as it was."""
+        src = h if h is not None else delta
+        n = src.shape[0] if rows is None else rows.numel()
+        dim = src.shape[1]
+        assert h is None or (h.is_contiguous() and h.dtype == torch.float32)
+        assert delta is None or (delta.is_contiguous() and delta.shape == src.shape)
+        for w in (delta_weight, weight):
+            assert w is None or (w.dtype == torch.float32 and w.is_contiguous() and w.numel() == dim)
+        assert out is None or (out.is_contiguous() and out.shape == (n, dim))
+        assert rows is None or (rows.dtype == torch.int32 and out is not None)
+        _check(self.lib, self.lib.fg_part_norm(
+            _ptr(h), int(fresh), _ptr(delta), _code(delta.dtype) if delta is not None else 0, _ptr(delta_weight),
+            _ptr(weight), _ptr(out), _code(out.dtype) if out is not None else 0, _ptr(rows), n, dim, int(parts),
+            float(eps), _stream()))
+        return out
+
     def linear_f32(self, x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
         """``x @ w.T`` in float32 whatever the serving type: ``w`` [N, K] float32, ``x`` [M, K] of either
         type (16-bit activations are widened as they are read); IEEE sums in ascending k."""
@@ -703,17 +728,18 @@ class Ops:
         return out
 
     # -- routed experts -----------------------------------------------------------------------------
-    def moe_logits(self, x: torch.Tensor, w: torch.Tensor, ctx=None) -> torch.Tensor:
-        """The router's logits ``x @ w.T`` in float32 whatever the serving type: ``w`` [E, K] float32,
-        ``x`` [T, K] of either type (16-bit activations are widened as they are read).  A warp a
-        token, sums in a fixed order: a token's logits do not depend on its batch.  Rows of padding
-        tokens (with ``ctx``) are left unwritten."""
+    def moe_logits(self, x: torch.Tensor, w: torch.Tensor, ctx=None, bias=None) -> torch.Tensor:
+        """The router's logits ``x @ w.T + bias`` in float32 whatever the serving type: ``w`` [E, K] and
+        ``bias`` [E] (or ``None``) float32, ``x`` [T, K] of either type (16-bit activations are widened as
+        they are read).  A block a token, sums in a fixed order: a token's logits do not depend on its
+        batch.  Rows of padding tokens (with ``ctx``) are left unwritten."""
         lib = moe()
         t, k = x.shape
         n = w.shape[0]
         assert w.dtype == torch.float32 and w.shape[1] == k and x.stride(1) == 1 and w.stride(1) == 1
+        assert bias is None or (bias.dtype == torch.float32 and bias.numel() == n and bias.is_contiguous())
         out = torch.empty((t, n), dtype=torch.float32, device=x.device)
-        _check(lib, lib.fg_moe_logits(_ptr(x), _code(x.dtype), x.stride(0), _ptr(w), w.stride(0), _ptr(out),
+        _check(lib, lib.fg_moe_logits(_ptr(x), _code(x.dtype), x.stride(0), _ptr(w), w.stride(0), _ptr(bias), _ptr(out),
                                       _ptr(ctx.req) if ctx is not None else None, t, n, k, _stream()))
         return out
 
@@ -728,22 +754,23 @@ class Ops:
         [T, top], weights float32 [T, top]); padding tokens get expert -1."""
         lib = moe()
         t, n = logits.shape
-        assert logits.dtype == torch.float32 and logits.is_contiguous()
+        assert logits.dtype == torch.float32 and logits.stride(1) == 1
         assert correction is None or (correction.dtype == torch.float32 and correction.numel() == n)
         ids = torch.empty((t, top), dtype=torch.int32, device=logits.device)
         weights = torch.empty((t, top), dtype=torch.float32, device=logits.device)
         if score != "softmax" or groups is not None or renorm_eps or weight_scale != 1.0:
             count, keep, group_top = groups if groups is not None else (0, 0, 0)
             _check(lib, lib.fg_moe_route_groups(
-                _ptr(logits), _ptr(correction), _ptr(ids), _ptr(weights), _ptr(ctx.req), t, n, int(top),
+                _ptr(logits), logits.stride(0), _ptr(correction), _ptr(ids), _ptr(weights), _ptr(ctx.req), t, n, int(top),
                 {"softmax": 0, "sigmoid": 1}[score], int(count), int(keep), int(group_top), int(renormalize),
                 float(renorm_eps), float(weight_scale), _stream()))
             return ids, weights
-        _check(lib, lib.fg_moe_route(_ptr(logits), _ptr(correction), _ptr(ids), _ptr(weights), _ptr(ctx.req), t, n,
-                                     int(top), int(renormalize), _stream()))
+        _check(lib, lib.fg_moe_route(_ptr(logits), logits.stride(0), _ptr(correction), _ptr(ids), _ptr(weights),
+                                     _ptr(ctx.req), t, n, int(top), int(renormalize), _stream()))
         return ids, weights
 
-    def moe_experts(self, x, ids, weights, w1, w3, w2, w13=None, act: Optional[str] = None) -> torch.Tensor:
+    def moe_experts(self, x, ids, weights, w1, w3, w2, w13=None, act: Optional[str] = None, shared=None,
+                    shared_gate=None) -> torch.Tensor:
         """``sum_k weights[t, k] * expert_{ids[t, k]}(x[t])`` with expert ``e`` the gated feed-forward
         ``w2[e] (silu(w1[e] x) * (w3[e] x))``; ``w1``, ``w3`` [E, F, K] (each expert's matrix contiguous,
         the experts a fixed stride apart: they may be the halves of ``w13`` [E, 2F, K]) and ``w2``
@@ -755,7 +782,10 @@ class Ops:
         products are the vendor's; gate and combine stay these kernels.
 
         ``w3 = None``: the experts have no gate, ``w2[e] act(w1[e] x)`` with ``act`` a key of
-        ``ACTIVATIONS`` (``w13`` is then ``w1`` itself, for the grouped product)."""
+        ``ACTIVATIONS`` (``w13`` is then ``w1`` itself, for the grouped product).
+
+        ``shared`` [T, K]: a further summand of every token; with ``shared_gate`` (float32 [T], strided) it
+        is multiplied by ``sigmoid(shared_gate[t])``.  Both join in the kernel that sums the experts."""
         lib = moe()
         t, k = x.shape
         n_experts, f, _ = w1.shape
@@ -817,8 +847,12 @@ class Ops:
                 _check(lib, lib.fg_moe_gemm(_ptr(mid), mid.stride(0), _ptr(w2), None, w2.stride(0), _ptr(y), y.stride(0),
                                             code, k, f, None, top, *tiles))
         out = torch.empty((t, k), dtype=x.dtype, device=x.device)
-        _check(lib, lib.fg_moe_combine(_ptr(y), y.stride(0), _ptr(weights), _ptr(pair_row), _ptr(out), out.stride(0),
-                                       _code(x.dtype), t, k, top, _stream()))
+        assert shared is None or (shared.shape == (t, k) and shared.dtype == x.dtype and shared.stride(1) == 1)
+        assert shared_gate is None or (shared is not None and shared_gate.dtype == torch.float32 and shared_gate.shape == (t,))
+        _check(lib, lib.fg_moe_combine(
+            _ptr(y), y.stride(0), _ptr(weights), _ptr(pair_row), _ptr(shared), shared.stride(0) if shared is not None else 0,
+            _ptr(shared_gate), shared_gate.stride(0) if shared_gate is not None else 0, _ptr(out), out.stride(0),
+            _code(x.dtype), t, k, top, _stream()))
         return out
 
     def linear(self, x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None,
@@ -975,7 +1009,8 @@ class Ops:
 
     def head_gate(self, x, gate, req, heads: int, head_dim: int) -> torch.Tensor:
         """``x[t, h, :] *= sigmoid(gate[t, h])`` in place (float32 arithmetic): ``x`` [T, heads * head_dim],
-        ``gate`` a row-strided view [T, heads] of the same type."""
+        ``gate`` a row-strided view [T, heads] of the same type.  ``head_dim = 1`` is the gate with a number
+        of its own for every column."""
         assert x.stride(1) == 1 and gate.stride(1) == 1 and x.dtype == gate.dtype and x.shape[1] == heads * head_dim
         _check(self.lib, self.lib.fg_head_gate(_ptr(x), x.stride(0), _ptr(gate), gate.stride(0), _code(x.dtype),
                                                _ptr(req), x.shape[0], heads, head_dim, _stream()))

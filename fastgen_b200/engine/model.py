@@ -18,6 +18,7 @@ from ..parts.base import (
     Block,
     CacheSpec,
     Embedder,
+    OpenStream,
     Part,
     StateSpec,
     WeightSpec,
@@ -67,9 +68,12 @@ def _build_embedder(args: ModelArgs) -> Embedder:
     return make_embedder(spec)
 
 
-def _collect_specs(args: ModelArgs, blocks: Sequence[Block], final_norm, embedder: Embedder) -> List[WeightSpec]:
+def _collect_specs(args: ModelArgs, blocks: Sequence[Block], final_norm, embedder: Embedder,
+                   embed_norm=None) -> List[WeightSpec]:
     specs: Dict[str, WeightSpec] = {}
     ordered = list(embedder.weight_specs())
+    if embed_norm is not None:
+        ordered.extend(embed_norm.weight_specs())
     for block in blocks:
         for part in block.parts():
             ordered.extend(part.weight_specs())
@@ -89,7 +93,8 @@ def _collect_specs(args: ModelArgs, blocks: Sequence[Block], final_norm, embedde
 
 def model_weight_specs(args: ModelArgs) -> List[WeightSpec]:
     """Every checkpoint tensor a model of this description needs, in a fixed order."""
-    return _collect_specs(args, _build_blocks(args), make_norm(args.final_norm), _build_embedder(args))
+    return _collect_specs(args, _build_blocks(args), make_norm(args.final_norm), _build_embedder(args),
+                          make_norm(args.embed_norm) if args.embed_norm is not None else None)
 
 
 class Model:
@@ -101,6 +106,7 @@ class Model:
         self.blocks = _build_blocks(args)
         self.final_norm = make_norm(args.final_norm)
         self.embedder = _build_embedder(args)
+        self.embed_norm = make_norm(args.embed_norm) if args.embed_norm is not None else None
         self.embedding: Optional[torch.Tensor] = None
         self.output: Optional[torch.Tensor] = None
         self.step_table: Optional[torch.Tensor] = None  # float32 [rows, dim]
@@ -110,7 +116,7 @@ class Model:
 
     # -- description -----------------------------------------------------------
     def weight_specs(self) -> List[WeightSpec]:
-        return _collect_specs(self.args, self.blocks, self.final_norm, self.embedder)
+        return _collect_specs(self.args, self.blocks, self.final_norm, self.embedder, self.embed_norm)
 
     def cache_specs(self) -> List[Optional[CacheSpec]]:
         return [self.blocks[e.layer].mixer.cache_spec() for e in self.args.schedule]
@@ -155,6 +161,8 @@ class Model:
             for part in block.parts():
                 add_part(part)
         add_part(self.final_norm)
+        if self.embed_norm is not None:
+            add_part(self.embed_norm)
         return total
 
     # -- weights -----------------------------------------------------------------
@@ -172,6 +180,8 @@ class Model:
         self.final_norm.bind(
             {local: tensors[name] for local, name in self.final_norm.names.items()}, self.ops
         )
+        if self.embed_norm is not None:
+            self.embed_norm.bind({local: tensors[name] for local, name in self.embed_norm.names.items()}, self.ops)
         if self.args.step_table_name is not None:
             # the vectors join the float32 residual sum: float32 whatever they were stored in
             self.step_table = tensors[self.args.step_table_name].float().contiguous()
@@ -251,6 +261,13 @@ class Model:
         self.embedder.forward(ctx, getattr(memories, "embedder_state", None), h)
         pending = None
         embed_part = None
+        if self.embed_norm is not None:
+            first = self.args.schedule[0]
+            if self.blocks[first.layer].opens_stream and self.pass_embed is None and first.step_row is None:
+                # the first block's kernel norms the embedding into the stream
+                h, pending = torch.empty_like(h), OpenStream(h, self.embed_norm)
+            else:
+                h = self.embed_norm.forward(h, out_dtype=torch.float32)
         if self.pass_embed is not None:
             # the embedder's output meets its half of the map once a step: that product is the same
             # before every pass

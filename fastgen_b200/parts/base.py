@@ -90,6 +90,9 @@ class Part:
 
 
 class Norm(Part):
+    """A norm.  A block that norms sub-layers' inputs calls ``forward`` and ``add_forward``; one that
+    norms their outputs only calls ``close``."""
+
     def _joined(self, h, total, rows):
         """For norms whose kernel does not take a :class:`ScaledSum`: add it to ``h`` with the kernel
         that does (needs ``self.ops``) and return ``None``; with ``rows`` (``h`` must stay as it
@@ -125,6 +128,21 @@ class Norm(Part):
                 return self.forward(h)
             h.add_(delta.to(h.dtype))
         return self.forward(h, rows=rows)
+
+
+    def close(self, h: torch.Tensor, delta, fresh: bool = False) -> torch.Tensor:
+        """``h += norm(delta)`` (32-bit sum, stored back; ``fresh``: ``h`` becomes it) and return the
+        stream itself as the next sub-layer reads it, in the compute dtype.
+
+        The default composes the steps; implementations may fuse them."""
+        if isinstance(delta, ScaledSum):
+            delta = self._joined(h, delta, True)
+        y = self.forward(delta, out_dtype=torch.float32)
+        if fresh:
+            h.copy_(y)
+        else:
+            h.add_(y)
+        return h.to(self.ops.act_dtype, copy=True)
 
 
 @dataclass
@@ -172,6 +190,15 @@ class NormedDelta:
 
     delta: torch.Tensor
     norm: Optional[Norm] = None
+
+
+@dataclass
+class OpenStream:
+    """The residual stream's first value on its way there: ``norm(source)`` (``source`` float32
+    [T, dim]).  Handed as ``pending`` to a first block that says ``opens_stream``."""
+
+    source: torch.Tensor
+    norm: Norm
 
 
 @dataclass
@@ -260,6 +287,9 @@ class Connection(Part):
 
 class Block:
     """Arrangement of a layer's parts around the residual stream."""
+
+    #: whether ``forward`` takes an :class:`OpenStream` as ``pending`` (it then writes ``h`` itself)
+    opens_stream = False
 
     def __init__(self, mixer: Mixer, mixer_norm: Norm, ffn: Optional[FeedForward], ffn_norm: Optional[Norm],
                  params=None, **extra: Part):

@@ -2,7 +2,9 @@
 
 from __future__ import annotations
 
-from .base import Block, NormedDelta, ScaledSum, register_block, split_pending
+import torch
+
+from .base import Block, NormedDelta, OpenStream, ScaledSum, register_block, split_pending
 
 
 class PreNormBlock(Block):
@@ -44,6 +46,39 @@ class SandwichBlock(Block):
         return h, NormedDelta(self.ffn.forward(f, ctx), self.extra.get("post_ffn_norm"))
 
 
+class PostNormBlock(Block):
+    """Norms on the sub-layers' outputs only: ``h = h + norm1(mixer(h)); h = h + norm2(ffn(h))`` with
+    ``norm1`` the ``mixer_norm`` and ``norm2`` the ``ffn_norm``.
+
+    A sub-layer reads the residual stream itself, in the compute dtype.  Its output is handed on with
+    the norm that closes it, so that one kernel (``Norm.close``) norms it, adds it to the stream and
+    stores what the next sub-layer reads.  A layer without a feed-forward ends after the mixer."""
+
+    opens_stream = True
+
+    def _read(self, h, pending):
+        if isinstance(pending, OpenStream):
+            return pending.norm.close(h, pending.source, fresh=True)
+        delta, norm = split_pending(pending)
+        if norm is not None:
+            return norm.close(h, delta)
+        ops = self.mixer_norm.ops
+        x = torch.empty(h.shape, dtype=ops.act_dtype, device=h.device)
+        total = ScaledSum.of(delta)
+        if len(total.terms) > 4 or len({t.dtype for t, _ in total.terms}) > 1:
+            total.add_into(h, ops)
+            total = ScaledSum([])
+        return ops.rmsnorm_sum(h, total.terms, None, 0.0, out=x, row=total.row)
+
+    def forward(self, h, pending, ctx, memory):
+        x = self._read(h, pending)
+        m = self.mixer.forward(x, ctx, memory)
+        if self.ffn is None:
+            return h, NormedDelta(m, self.mixer_norm)
+        x = self.mixer_norm.close(h, m)
+        return h, NormedDelta(self.ffn.forward(x, ctx), self.ffn_norm)
+
+
 class StreamsBlock(Block):
     """Pre-norm sub-layers on several residual streams: ``h`` is [T, streams, dim] and every
     sub-layer reads and writes it through a connection of its own, the extra parts
@@ -80,4 +115,5 @@ class ParallelBlock(Block):
 register_block("prenorm", PreNormBlock)
 register_block("parallel", ParallelBlock)
 register_block("streams", StreamsBlock)
+register_block("postnorm", PostNormBlock)
 register_block("sandwich", SandwichBlock)

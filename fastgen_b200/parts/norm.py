@@ -7,7 +7,7 @@ from typing import List
 import torch
 
 from .base import Norm, ScaledSum, StreamUpdate, WeightSpec, register_norm
-from .params import DynamicTanhParams, LayerNormParams, RMSNormParams
+from .params import DynamicTanhParams, LayerNormParams, PartRMSNormParams, RMSNormParams
 
 
 class RMSNorm(Norm):
@@ -147,6 +147,50 @@ class LayerNorm(Norm):
         return self.streams_forward(h, update=update, rows=rows)
 
 
+class PartRMSNorm(Norm):
+    """RMS norm in equal consecutive parts of a row, in float32 (see :class:`PartRMSNormParams`).
+
+    As the norm that closes a sub-layer it adds the normed output to the residual stream and hands out
+    the sum as the next sub-layer reads it in one kernel (``close``)."""
+
+    params: PartRMSNormParams
+
+    def weight_specs(self) -> List[WeightSpec]:
+        return [WeightSpec(self.names["weight"], (self.params.dim,), ("ones",))]
+
+    def bind(self, tensors, ops) -> None:
+        self.ops = ops
+        # a small vector: float32 whatever it was stored in (the arithmetic is float32)
+        self.weight = tensors["weight"].float().contiguous()
+
+    def _out(self, x, rows, out_dtype=None):
+        n = x.shape[0] if rows is None else rows.numel()
+        return torch.empty((n, x.shape[1]), dtype=out_dtype or self.ops.act_dtype, device=x.device)
+
+    def forward(self, x, out_dtype=None, rows=None):
+        p = self.params
+        return self.ops.part_norm(p.parts, p.eps, delta=x, delta_weight=self.weight, out=self._out(x, rows, out_dtype),
+                                  rows=rows)
+
+    def close(self, h, delta, fresh=False):
+        p = self.params
+        if isinstance(delta, ScaledSum):
+            delta = self._joined(h, delta, True)
+        return self.ops.part_norm(p.parts, p.eps, h=h, delta=delta, delta_weight=self.weight, out=self._out(h, None),
+                                  fresh=fresh)
+
+    def add_forward(self, h, delta, rows=None, delta_norm=None):
+        p = self.params
+        if isinstance(delta, ScaledSum):
+            delta = self._joined(h, delta, True if delta_norm is not None else rows)
+        same = isinstance(delta_norm, PartRMSNorm) and (delta_norm.params.parts, delta_norm.params.eps) == (p.parts, p.eps)
+        if delta is not None and not same:
+            return super().add_forward(h, delta, rows=rows, delta_norm=delta_norm)
+        return self.ops.part_norm(p.parts, p.eps, h=h, delta=delta, weight=self.weight, out=self._out(h, rows), rows=rows,
+                                  delta_weight=delta_norm.weight if delta is not None else None)
+
+
 register_norm("rmsnorm", RMSNorm)
+register_norm("part_rmsnorm", PartRMSNorm)
 register_norm("layernorm", LayerNorm)
 register_norm("dynamic_tanh", DynamicTanh)

@@ -197,6 +197,20 @@ class RMSNormParams:
 
 
 @dataclass(frozen=True)
+class PartRMSNormParams:
+    """An RMS norm in ``parts`` equal consecutive parts of a row, each divided by its own
+    ``sqrt(mean(part^2) + eps)``, then one weight over the whole row."""
+
+    dim: int
+    eps: float
+    parts: int = 1
+
+    def __post_init__(self) -> None:
+        if self.parts < 1 or self.dim % self.parts:
+            raise ValueError(f"{self.dim} columns cannot be normed in {self.parts} equal parts")
+
+
+@dataclass(frozen=True)
 class DenseMLPParams:
     """Dense feed-forward ``down(act(up x))`` without a gate; ``act`` is ``"gelu_erf"`` (the
     exact GELU), ``"gelu_tanh"`` or ``"relu2"`` (the square of ReLU)."""
@@ -303,27 +317,35 @@ class Mamba2Params:
 class LatentAttentionParams:
     """Causal softmax attention whose keys and values are linear maps of a cached latent.
 
-    Queries come through a latent of ``q_rank`` numbers (RMS-normed); a head's query and key have
-    ``head_dim`` unrotated and ``rot_dim`` rotated dimensions (``position`` is the ``PartSpec`` of
-    the rotation of those), its value ``v_head_dim``.  A token caches ``kv_rank`` latent numbers
-    (RMS-normed) and one rotated key part that all heads share.  ``own_cache`` false: the layer
-    has no latent projection and reads the entries another layer caches.  ``gate``: every head's
-    output is multiplied by the sigmoid of a projection of the mixer's input."""
+    Queries come through a latent of ``q_rank`` numbers (RMS-normed), or with ``q_rank`` ``None``
+    straight from the mixer's input; a head's query and key have ``head_dim`` unrotated and ``rot_dim``
+    rotated dimensions (``position`` is the ``PartSpec`` of the rotation of those; 0: no rotated part),
+    its value ``v_head_dim``.  A token caches ``kv_rank`` latent numbers (RMS-normed) and one rotated
+    key part that all heads share.  ``own_cache`` false: the layer has no latent projection and reads
+    the entries another layer caches.  ``gate``: the heads' outputs are multiplied by the sigmoid of a
+    projection of the mixer's input that has a number per head (``"head"``) or one per value dimension
+    of every head (``"value"``); ``None``: no gate.  ``rot_layout`` is the checkpoint's pairing of the
+    rotated dimensions, as ``AttentionParams.qk_layout``."""
 
     dim: int
     n_heads: int
     head_dim: int
     rot_dim: int
     v_head_dim: int
-    q_rank: int
+    q_rank: Optional[int]
     kv_rank: int
     softmax_scale: float
     eps: float
     position: object
     own_cache: bool = True
-    gate: bool = True
+    gate: Optional[str] = "head"
+    rot_layout: str = "adjacent"
 
     def __post_init__(self) -> None:
+        if self.gate not in (None, "head", "value"):
+            raise ValueError(f"gate must be None, 'head' or 'value', got {self.gate!r}")
+        if self.rot_layout not in ("adjacent", "half_split"):
+            raise ValueError(f"rot_layout must be 'adjacent' or 'half_split', got {self.rot_layout!r}")
         if self.rot_dim % 2:
             raise ValueError(f"the rotated part has {self.rot_dim} dimensions: a rotation needs pairs")
         if not 1 <= self.kv_rank <= 512:
@@ -406,10 +428,18 @@ class RoutedExpertsParams:
     act: str = "silu_gate"
     #: a ``PartSpec`` of a feed-forward that every token also passes and whose output is added
     shared: Optional[object] = None
+    #: the shared feed-forward's output is multiplied by the sigmoid of one number per token, a projection
+    #: of the input (tensor ``shared_gate`` [1, dim], float32 arithmetic as the router's)
+    shared_gate: bool = False
+    #: the router's logits have a bias (tensor ``router_bias`` [experts]) that counts in the choice and in
+    #: the weights
+    router_bias: bool = False
 
     def __post_init__(self) -> None:
         if not 1 <= self.top <= self.n_experts:
             raise ValueError(f"a token cannot use {self.top} of {self.n_experts} experts")
+        if self.shared_gate and self.shared is None:
+            raise ValueError("a gate of the shared expert without a shared expert")
         if self.n_experts > 256:
             raise ValueError(f"the router takes up to 256 experts, got {self.n_experts}")
         if self.score not in ("softmax", "sigmoid"):

@@ -23,8 +23,10 @@ class RoutedExperts(FeedForward):
 
     Options of the parameters: sigmoid scores instead of a softmax; a choice that is limited to the
     experts of the best groups of neighbours; a small number added to the sum that renormalises; a
-    factor on the weights; experts without a gate, ``w2_e(act(w3_e x))``; a shared feed-forward that every
-    token passes and whose output is added (the result is then a sum that the next norm's kernel forms).
+    factor on the weights; a bias of the router's logits; experts without a gate, ``w2_e(act(w3_e x))``; a
+    shared feed-forward that every token passes and whose output is added (the result is then a sum that
+    the next norm's kernel forms), or multiplied by the sigmoid of one number per token and added (the
+    number is one more row of the router's product, and the kernel that sums the experts adds it).
     """
 
     params: RoutedExpertsParams
@@ -51,7 +53,7 @@ class RoutedExperts(FeedForward):
             if local in ("w1", "w2", "w3"):
                 for e in range(self.params.n_experts):
                     flat[f"{local}.{e}"] = name.format(e)
-            elif local != "correction" or self.params.correction:
+            elif getattr(self.params, local, True):  # "correction", "router_bias", "shared_gate": where asked for
                 flat[local] = name
         if self.params.shared is not None:
             for local, name in dict(self.params.shared.names).items():
@@ -63,6 +65,10 @@ class RoutedExperts(FeedForward):
         specs = [WeightSpec(n["router"], (p.n_experts, p.dim), ("normal", 0.5))]
         if p.correction:
             specs.append(WeightSpec(n["correction"], (p.n_experts,), ("normal", 0.05)))
+        if p.router_bias:
+            specs.append(WeightSpec(n["router_bias"], (p.n_experts,), ("normal", 0.5)))
+        if p.shared_gate:
+            specs.append(WeightSpec(n["shared_gate"], (1, p.dim), ("normal", 0.1)))
         for e in range(p.n_experts):
             if self.gated:
                 specs.append(WeightSpec(n["w1"].format(e), (p.ffn_dim, p.dim)))
@@ -89,20 +95,31 @@ class RoutedExperts(FeedForward):
             self.w3, self.w2 = None, stack("w2")
         if self.shared is not None:
             self.shared.bind({local: tensors["shared." + local] for local in self.shared.names}, ops)
-        self.router = tensors["router"].float().contiguous()
+        router = tensors["router"].float()
+        bias = tensors["router_bias"].float() if p.router_bias else None
+        if p.shared_gate:
+            # one more row of the router's product (without a bias)
+            router = torch.cat([router, tensors["shared_gate"].float()], dim=0)
+            bias = torch.cat([bias, bias.new_zeros(1)]) if bias is not None else None
+        self.router = router.contiguous()
+        self.router_bias = bias.contiguous() if bias is not None else None
         self.correction = tensors["correction"].float().contiguous() if p.correction else None
 
     def forward(self, x, ctx):
         p, ops = self.params, self.ops
-        logits = ops.moe_logits(x, self.router, ctx)
+        logits = ops.moe_logits(x, self.router, ctx, bias=self.router_bias)
+        gate = logits[:, p.n_experts] if p.shared_gate else None
+        logits = logits[:, : p.n_experts]
         groups = (*p.groups, p.group_top) if p.groups is not None else None
         ids, weights = ops.moe_route(logits, self.correction, p.top, ctx, renormalize=p.renormalize, score=p.score,
                                      groups=groups, renorm_eps=p.renorm_eps, weight_scale=p.weight_scale)
-        out = ops.moe_experts(x, ids, weights, self.w1, self.w3, self.w2, self.w13,
-                              act=None if self.gated else p.act)
-        if self.shared is None:
+        shared = self.shared.forward(x, ctx) if self.shared is not None else None
+        gated = gate is not None  # (then the experts' sum takes the shared output in)
+        out = ops.moe_experts(x, ids, weights, self.w1, self.w3, self.w2, self.w13, act=None if self.gated else p.act,
+                              shared=shared if gated else None, shared_gate=gate)
+        if shared is None or gated:
             return out
-        return ScaledSum([(out, 1.0), (self.shared.forward(x, ctx), 1.0)])
+        return ScaledSum([(out, 1.0), (shared, 1.0)])
 
 
 register_feed_forward("routed_experts", RoutedExperts)
