@@ -1,6 +1,6 @@
 """Throughput of one design beside another at equal size, step by step and kernel by kernel.
 
-``bench.py --design sinorax|zeladra|tanupel|palulorn`` runs this: prefill and decode throughput of a model of that
+``bench.py --design sinorax|zeladra|tanupel|palulorn|kuvusun`` runs this: prefill and decode throughput of a model of that
 design at a few sizes that resemble a real model's layers (random weights), beside a Llama-shaped model of
 the same width, heads, head size, number of layers and number of parameters a layer, and the
 time of each kernel family of the two designs at those sizes with its fraction of the roofline
@@ -56,10 +56,12 @@ def sinorax_config(width, layers, heads, kv, head_dim, ffn, vocab, window, kinds
                 embedding=dict(bigram=dict(buckets=65521, mul_prev=1000003, mul_cur=31)), layers=out)
 
 
-def zeladra_config(width, layers, heads, kv, head_dim, ffn, vocab, window) -> dict:
+def zeladra_config(width, layers, heads, kv, head_dim, ffn, vocab, window,
+                   kinds=("latent_attention", "mamba2", "attention"), streams=2) -> dict:
     """Latent attention, the state-space mixer and windowed attention that keeps the first four
     positions, in turn (every second latent layer reads the first one's cache), on two residual
-    streams; every layer has the gated feed-forward of the Llama shape."""
+    streams; every layer has the gated feed-forward of the Llama shape.  (``kinds``: another order, say
+    latent layers only; ``streams`` ``None``: the one ordinary stream.)"""
     latent = dict(heads=heads, dim=head_dim, rot_dim=head_dim // 2, vdim=head_dim, q_rank=width * 3 // 4,
                   kv_rank=4 * head_dim, scale=(head_dim * 3 // 2) ** -0.5,
                   rot=dict(dims=head_dim // 2, base=500000.0, scaling=dict(factor=4.0, original=8192, fast=32.0, slow=1.0)))
@@ -68,16 +70,18 @@ def zeladra_config(width, layers, heads, kv, head_dim, ffn, vocab, window) -> di
                rot=dict(dims=head_dim, base=500000.0), mask=dict(size=window, keep_first=4))
     out, first_latent = [], None
     for i in range(layers):
-        kind = ("latent_attention", "mamba2", "attention")[i % 3]
+        kind = kinds[i % len(kinds)]
         mixer = dict({"latent_attention": latent, "mamba2": ssm, "attention": att}[kind])
         if kind == "latent_attention":
             if first_latent is None:
                 first_latent = i
-            elif (i // 3) % 2 == 1:
+            elif (i // len(kinds)) % 2 == 1:
                 mixer["kv_from"] = first_latent
         out.append(dict(type=kind, mixer=mixer, mlp=dict(kind="dense", ff=ffn)))
-    return dict(architecture="Zeladra", vocab=vocab, width=width, norm=dict(eps=1e-5), embedding=dict(scale=1.0),
-                streams=2, layers=out)
+    cfg = dict(architecture="Zeladra", vocab=vocab, width=width, norm=dict(eps=1e-5), embedding=dict(scale=1.0), layers=out)
+    if streams is not None:
+        cfg["streams"] = streams
+    return cfg
 
 
 def tanupel_config(width, layers, heads, kv, head_dim, ffn, vocab, window=None, experts=8, top=2) -> dict:
@@ -125,6 +129,25 @@ def palulorn_config(width, layers, heads, kv, head_dim, ffn, vocab, window=1024,
     out = [dict(type=mixers[i % 3][0], mixer=dict(mixers[i % 3][1]), mlp=dict(routed)) for i in range(layers)]
     return dict(architecture="Palulorn", vocab=vocab, width=width, norm=dict(eps=1e-5), embedding=dict(scale=1.0),
                 loop=dict(start=0, stop=layers, times=1), layers=out)
+
+
+def kuvusun_config(width, layers, heads, kv, head_dim, ffn, vocab, window=None, experts=8, top=2) -> dict:
+    """Latent attention with a turned part and an output gate, and latent attention without positions
+    (queries through a latent), in turn; every second layer of the first kind reads the cache of the one
+    before it.  The first layer's feed-forward is dense (a squared ReLU, half as wide again as the gated
+    one), the others are routed: ``experts`` gated experts of ``ffn / experts`` rows and a gated shared one."""
+    turned = dict(heads=heads, dim=head_dim, rot_dim=head_dim // 2, vdim=head_dim, kv_rank=4 * head_dim,
+                  scale=(head_dim * 3 // 2) ** -0.5, rot=dict(dims=head_dim // 2, base=500000.0))
+    plain = dict(heads=heads, dim=head_dim, vdim=head_dim, q_rank=width * 3 // 4, kv_rank=4 * head_dim, scale=head_dim ** -0.5)
+    routed = dict(kind="moe", expert=dict(ff=ffn // experts), router=dict(experts=experts, top=top), shared=dict(ff=ffn // experts))
+    out = []
+    for i in range(layers):
+        mixer = dict(turned if i % 2 == 0 else plain)
+        if i % 4 == 2:
+            mixer["kv_from"] = i - 2
+        out.append(dict(type="latent_attention_2" if i % 2 == 0 else "latent_attention", mixer=mixer,
+                        mlp=dict(kind="dense", ff=ffn * 3 // 2) if i == 0 else dict(routed)))
+    return dict(architecture="Kuvusun", vocab=vocab, width=width, norm=dict(eps=1e-5, groups=8), layers=out)
 
 
 class Timer:
@@ -430,7 +453,7 @@ def _latent_attention_times(cfg, device, timer: Timer, layer: int) -> Dict[str, 
     def run(t, ctx):
         qa = torch.randn(H, t, R, generator=gen).to(device, torch.bfloat16)
         q = torch.randn(t, H, d + r, generator=gen).to(device, torch.bfloat16)
-        gate = torch.randn(t, H, generator=gen).to(device, torch.bfloat16)
+        gate = torch.randn(t, H, generator=gen).to(device, torch.bfloat16) if p.gate == "head" else None
         o = torch.empty_like(qa)
         return timer.us(lambda: engine.ops.latent_attention(qa, q[:, :, d:], o, gate, memory, ctx, H, R, r, p.softmax_scale))
 
@@ -840,9 +863,147 @@ def palulorn_kernel_table(size, device, peaks) -> Dict[str, dict]:
     return table
 
 
+def kuvusun_kernel_table(size, device, peaks) -> Dict[str, dict]:
+    """The kernels of the Kuvusun design alone at one size, each beside the like kernel of the closest
+    model where there is one (Zeladra's latent attention, Tanupel's routed experts, the Llama shape's norm
+    and gated feed-forward): microseconds and the fraction of the roofline."""
+    from ..cache import LayerMemory
+    from ..csrc.ops import Ops
+    from ..engine.step import StepContext
+    from ..parts.base import StreamUpdate
+
+    width, _layers, heads, kv, head_dim, ffn, vocab, window = size
+    ops = Ops(torch.bfloat16, device)
+    timer = Timer(device)
+    gen = torch.Generator().manual_seed(SEED)
+    hbm, tensor = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    table: Dict[str, dict] = {}
+
+    def bw(name, us, nbytes):
+        table[name] = dict(us=round(us, 1), gbs=round(nbytes / (us * 1e-6) / 1e9, 1), hbm_frac=round(nbytes / (us * 1e-6) / hbm, 3))
+
+    def rand(*shape, dtype=torch.bfloat16):
+        return torch.randn(*shape, generator=gen).to(device, dtype)
+
+    def context(t, n_seqs):
+        ctx = StepContext(device)
+        per = t // n_seqs
+        ctx.req = torch.arange(n_seqs, dtype=torch.int32, device=device).repeat_interleave(per)
+        ctx.pos = torch.arange(per, dtype=torch.int32, device=device).repeat(n_seqs)
+        ctx.seq_slot = torch.arange(n_seqs, dtype=torch.int32, device=device)
+        ctx.seq_start = torch.arange(0, t + 1, per, dtype=torch.int32, device=device)
+        ctx.n_tokens, ctx.n_seqs = t, n_seqs
+        return ctx
+
+    few = lambda t: t == DECODE_BATCH  # few tokens: time the captured launches (device time, not the host's)
+    cfg = kuvusun_config(*size)
+    turned, plain = cfg["layers"][0]["mixer"], cfg["layers"][1]["mixer"]
+    R, r, d, dv = turned["kv_rank"], turned["rot_dim"], turned["dim"], turned["vdim"]
+    for t in (PREFILL_TOKENS, DECODE_BATCH):
+        h, delta = rand(t, width, dtype=torch.float32), rand(t, width)
+        out = torch.empty(t, width, dtype=torch.bfloat16, device=device)
+        w, b, wb = rand(width, dtype=torch.float32), rand(width, dtype=torch.float32), rand(width)
+        nbytes = t * width * (4 + 4 + 2 + 2)
+        bw(f"norm+sum t={t}: rmsnorm in 8 parts of the output, sum", timer.us(lambda: ops.part_norm(
+            8, 1e-5, h=h, delta=delta, delta_weight=w, out=out), graph=few(t)), nbytes)
+        bw(f"norm+sum t={t}: rmsnorm in 8 parts of the output, sum, norm of the sum (the model's end)", timer.us(lambda: ops.part_norm(
+            8, 1e-5, h=h, delta=delta, delta_weight=w, weight=b, out=out), graph=few(t)), nbytes)
+        bw(f"norm+sum t={t}: layer norm (sum, norm; zeladra on one stream)", timer.us(lambda: ops.stream_norm(
+            h.view(t, 1, width), w, b, 1e-5, out, update=StreamUpdate(delta)), graph=few(t)), nbytes)
+        bw(f"norm+sum t={t}: rmsnorm (sum, norm; llama)", timer.us(lambda: ops.rmsnorm(h, wb, 1e-5, out=out, delta=delta), graph=few(t)), nbytes)
+
+        # what a mixer launches around its attention
+        ctx = context(t, 1 if t == PREFILL_TOKENS else t)
+        cols = heads * (d + r) + heads * dv + R + r
+        proj = rand(t, cols)
+        freqs = torch.rand(r // 2, generator=gen).to(device)
+        bw(f"turned part of the queries t={t} (halves of the projection's rows)", timer.us(lambda: ops.rotate_part(
+            proj[:, : heads * (d + r)], ctx, freqs, 1.0, heads, d + r, d, r), graph=few(t)), t * heads * r * 4)
+        o, gate = rand(t, heads * dv), proj[:, heads * (d + r) : heads * (d + r) + heads * dv]
+        bw(f"output gate t={t}: a number a column", timer.us(lambda: ops.head_gate(o, gate, ctx.req, heads * dv, 1), graph=few(t)),
+           t * heads * dv * 6)
+        x13, g = rand(t, 2 * ffn), torch.empty(t, ffn, dtype=torch.bfloat16, device=device)
+        bw(f"activation t={t}: silu gate [t, 2 f] -> [t, f] (llama)", timer.us(lambda: ops.silu_gate(x13, g, 8), graph=few(t)), t * ffn * 6)
+        c_w = rand(plain["q_rank"], dtype=torch.float32)
+        down = rand(t, plain["q_rank"] + R)
+        bw(f"norm of the query latent t={t}", timer.us(lambda: ops.rms_rows(down[:, : plain["q_rank"]], c_w, 1e-5), graph=few(t)),
+           t * plain["q_rank"] * 4)
+        pages = -(-t // PAGE)
+        n_seqs = ctx.n_seqs
+        bt = torch.arange(n_seqs * pages, dtype=torch.int32, device=device).view(n_seqs, pages)
+        for what, rot in (("latent and turned key part", r), ("latent", 0)):
+            pool = torch.zeros(n_seqs * pages, 1, PAGE, R + rot, dtype=torch.bfloat16, device=device)
+            mem = LayerMemory(k_pages=pool, v_pages=None, block_table=bt, page_size=PAGE)
+            nw = rand(R, dtype=torch.float32)
+            bw(f"cache entry t={t}: {what}", timer.us(lambda: ops.latent_entry_write(
+                proj[:, cols - R - rot :], nw, 1e-5, freqs, 1.0, mem, ctx, R, rot), graph=few(t)), t * (R + rot) * 4)
+
+    # routed experts with a gated shared one beside Tanupel's
+    E, top, f = 8, 2, ffn // 8
+    w13, w2 = rand(E, 2 * f, width), rand(E, width, f)
+    router, more, bias = rand(E, width, dtype=torch.float32), rand(E + 1, width, dtype=torch.float32), rand(E + 1, dtype=torch.float32)
+    for t in (PREFILL_TOKENS, DECODE_BATCH):
+        x, shared = rand(t, width), rand(t, width)
+        ctx = context(t, 1)
+        touched = min(E, t * top)
+        for name, weights_of, b, kw in (("kuvusun: bias, one more row, shared expert's gate", more, bias, True), ("tanupel", router, None, False)):
+            logits = ops.moe_logits(x, weights_of, bias=b)
+            chosen = logits[:, :E]
+            route = lambda: ops.moe_route(chosen, None, top, ctx, renormalize=kw)
+            ids, weights = route()
+            extra = dict(shared=shared, shared_gate=logits[:, E]) if kw else {}
+            us = timer.us(lambda: ops.moe_experts(x, ids, weights, w13[:, :f], w13[:, f:], w2, w13, **extra), graph=few(t))
+            flops = 6 * t * top * f * width
+            table[f"routed experts t={t}: {top} of {E} experts of {f} rows ({name})"] = dict(
+                router_logits_us=round(timer.us(lambda: ops.moe_logits(x, weights_of, bias=b), graph=few(t)), 1),
+                choice_us=round(timer.us(route, graph=few(t)), 1), experts_us=round(us, 1),
+                experts_tflops=round(flops / (us * 1e-6) / 1e12, 1), experts_tensor_frac=round(flops / (us * 1e-6) / tensor, 3),
+                experts_hbm_frac=round(touched * 3 * f * width * 2 / (us * 1e-6) / hbm, 3))
+
+    small = (width, 4, heads, kv, head_dim, ffn, 1024)
+    kz = kuvusun_config(*small)
+    zz = zeladra_config(*small, window, kinds=("latent_attention",), streams=None)
+    for name, c, layer in (("kuvusun, turned part", kz, 0), ("kuvusun, no positions", kz, 1), ("zeladra", zz, 0)):
+        row = _latent_attention_times(c, device, timer, layer)
+        row["prefill_tensor_frac"] = round(row["prefill_tflops"] * 1e12 / tensor, 3)
+        row["decode_hbm_frac"] = round(row["decode_gbs"] * 1e9 / hbm, 3)
+        table[f"attention over latents ({name}; causal)"] = row
+    row = _attention_times(llama_config(*small), device, timer, 0, None, heads, kv, head_dim)
+    row["prefill_tensor_frac"] = round(row["prefill_tflops"] * 1e12 / tensor, 3)
+    row["decode_hbm_frac"] = round(row["decode_gbs"] * 1e9 / hbm, 3)
+    table["attention softmax (llama, causal)"] = row
+    # whole mixers and feed-forwards (projections included)
+    table["mixer latent attention, turned part and gate (kuvusun; whole mixer)"] = _mixer_times(kz, device, timer, 0)
+    table["mixer latent attention, no positions (kuvusun; whole mixer)"] = _mixer_times(kz, device, timer, 1)
+    table["mixer latent attention (zeladra; whole mixer)"] = _mixer_times(zz, device, timer, 0)
+    table["mixer attention (llama, causal; whole mixer)"] = _mixer_times(llama_config(*small), device, timer, 0)
+    table["feed-forward (kuvusun: squared ReLU, dense; whole)"] = _mixer_times(kz, device, timer, 0, pick=lambda b: b.ffn)
+    table["feed-forward (kuvusun: routed and shared experts; whole)"] = _mixer_times(kz, device, timer, 1, pick=lambda b: b.ffn)
+    table["feed-forward (tanupel: routed experts; whole)"] = _mixer_times(tanupel_config(*small), device, timer, 2, pick=lambda b: b.ffn)
+    table["feed-forward (llama, gated; whole)"] = _mixer_times(llama_config(*small), device, timer, 0, pick=lambda b: b.ffn)
+    return table
+
+
 def run(sizes: List[str], peaks: dict, kernels: bool = True, design: str = "sinorax") -> dict:
     device = torch.device("cuda:0")
     torch.cuda.set_device(device)
+    if design == "kuvusun":
+        out = {"metric": "prefill and decode tokens/s of Kuvusun beside Zeladra (latent layers only) and a Llama-shaped model of equal size (bf16, random weights)",
+               "unit": "tokens/s", "dtype": "bf16", "data": "synthetic (random weights, uniform random token ids)",
+               "config": dict(prefill_tokens=PREFILL_TOKENS, decode_batch=DECODE_BATCH, decode_context=DECODE_CONTEXT, page=PAGE,
+                              l2="flushed before every timed kernel; model steps stream all weights"),
+               "peaks": peaks, "sizes": {}}
+        for name in sizes:
+            size = SIZES[name]
+            entry = dict(width=size[0], layers=size[1], heads=size[2], kv_heads=size[3], head_dim=size[4], swiglu_ffn=size[5],
+                         vocab=size[6], kv_rank=4 * size[4], rot_dim=size[4] // 2, experts=8, top=2, expert_ffn=size[5] // 8)
+            entry["kuvusun"] = model_throughput(kuvusun_config(*size), device)
+            entry["zeladra"] = model_throughput(zeladra_config(*size, kinds=("latent_attention",), streams=None), device)
+            entry["llama"] = model_throughput(llama_config(*size[:7]), device)
+            if kernels:
+                entry["kernels"] = kuvusun_kernel_table(size, device, peaks)
+            out["sizes"][name] = entry
+        return out
     if design == "palulorn":
         out = {"metric": "prefill and decode tokens/s of Palulorn beside Tanupel and a Llama-shaped model of equal size (bf16, random weights)",
                "unit": "tokens/s", "dtype": "bf16", "data": "synthetic (random weights, uniform random token ids)",

@@ -178,3 +178,16 @@ def greedy(config, tensors, prompt, n_new: int):
         out.append(tok)
         seq.append(tok)
     return out
+
+
+def read_model(model_dir, dtype=DT):
+    """``(config, tensors)`` of a model folder."""
+    import json
+    from pathlib import Path
+
+    from safetensors.torch import load_file
+
+    with open(Path(model_dir) / "config.json") as f:
+        config = json.load(f)
+    tensors = {k: v.to(dtype) for k, v in load_file(str(Path(model_dir) / "model.safetensors")).items()}
+    return config, tensors
