@@ -14,48 +14,149 @@
 // order of a row's sums depends on its own position only.
 #include "common.cuh"
 
-// ---- rotation of a part of each head ------------------------------------------------------------
-// x[t, head, offset + 2i], x[t, head, offset + 2i + 1] turn by pos[t] * freqs[i]; cosine and sine
-// are both multiplied by `magnitude`.  Angles are float32 products, sincosf is the precise one.
+// ---- what runs on the projections of a step's tokens ----------------------------------------------------
+// Three pieces, each one block's work on one token: the rotation of a part of every head of the queries,
+// the RMS norm of the query latent, and the cache entry.  Each has a kernel of its own, and
+// latent_prepare_kernel runs the entry and one piece of the query side as one launch.
+
+// Columns of a row as eight at a time where its address and width allow 16-byte loads (BF16 rows).
 template <typename T>
-__global__ void rotate_part_kernel(T* x, long stride, const int* __restrict__ pos, const int* __restrict__ req,
-                                   const float* __restrict__ freqs, float magnitude, int n_heads, int head_size,
-                                   int offset, int rot_dims) {
-  const int t = blockIdx.x;
-  if (req[t] < 0) return;
-  const float p = (float)pos[t];
+__device__ __forceinline__ bool rows_by_eight(const T*, int) {
+  return false;
+}
+template <>
+__device__ __forceinline__ bool rows_by_eight<__nv_bfloat16>(const __nv_bfloat16* p, int dim) {
+  return dim % 8 == 0 && ((uintptr_t)p & 15) == 0;
+}
+
+// sum of squares of row[0 .. dim), over the block (128 threads)
+template <typename T>
+__device__ __forceinline__ float row_squares(const T* row, int dim, float* scratch) {
+  float ss = 0.f;
+  if (rows_by_eight<T>(row, dim)) {
+#pragma unroll 4
+    for (int d = threadIdx.x * 8; d < dim; d += blockDim.x * 8) {
+      const uint4 raw = *reinterpret_cast<const uint4*>(row + d);
+      const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float2 f = __bfloat1622float2(h[i]);
+        ss = fmaf(f.x, f.x, ss);
+        ss = fmaf(f.y, f.y, ss);
+      }
+    }
+  } else {
+#pragma unroll 4
+    for (int d = threadIdx.x; d < dim; d += blockDim.x) {
+      const float v = to_f32<T>(row[d]);
+      ss = fmaf(v, v, ss);
+    }
+  }
+  return block_sum(ss, scratch);
+}
+
+// out[d] = row[d] * rstd * w[d]
+template <typename T>
+__device__ __forceinline__ void write_normed(const T* row, float rstd, const float* __restrict__ w, T* out, int dim) {
+  if (rows_by_eight<T>(row, dim) && rows_by_eight<T>(out, dim) && ((uintptr_t)w & 15) == 0) {
+    for (int d = threadIdx.x * 8; d < dim; d += blockDim.x * 8) {
+      const uint4 raw = *reinterpret_cast<const uint4*>(row + d);
+      const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+      const float4 w0 = *reinterpret_cast<const float4*>(w + d), w1 = *reinterpret_cast<const float4*>(w + d + 4);
+      const float wv[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
+      uint4 o;
+      __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&o);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float2 f = __bfloat1622float2(h[i]);
+        o2[i] = __floats2bfloat162_rn(f.x * rstd * wv[2 * i], f.y * rstd * wv[2 * i + 1]);
+      }
+      *reinterpret_cast<uint4*>(out + d) = o;
+    }
+  } else {
+    for (int d = threadIdx.x; d < dim; d += blockDim.x) out[d] = from_f32<T>(to_f32<T>(row[d]) * rstd * w[d]);
+  }
+}
+
+template <typename T>
+__device__ __forceinline__ void norm_row(const T* row, const float* __restrict__ w, float eps, T* out, int dim,
+                                         float* scratch) {
+  const float ss = row_squares<T>(row, dim, scratch);
+  write_normed<T>(row, 1.f / sqrtf(ss / (float)dim + eps), w, out, dim);
+}
+
+// Angles are float32 products, sincosf is the precise one; cosine and sine times `magnitude`.
+__device__ __forceinline__ void angle(float p, float freq, float magnitude, float& sn, float& cs) {
+  sincosf(p * freq, &sn, &cs);
+  sn *= magnitude;
+  cs *= magnitude;
+}
+
+// x[head, offset + 2i], x[head, offset + 2i + 1] of one token turn by p * freqs[i]
+template <typename T>
+__device__ __forceinline__ void turn_heads(T* x, float p, const float* __restrict__ freqs, float magnitude, int n_heads,
+                                           int head_size, int offset, int rot_dims) {
   const int pairs = rot_dims / 2;
+  // with a number of pairs that divides the block a thread meets one pair only: one sine and cosine
+  const bool one = blockDim.x % pairs == 0;
+  float sn = 0.f, cs = 1.f;
+  if (one) angle(p, freqs[threadIdx.x % pairs], magnitude, sn, cs);
   for (int i = threadIdx.x; i < n_heads * pairs; i += blockDim.x) {
     const int h = i / pairs, j = i - h * pairs;
-    float sn, cs;
-    sincosf(p * freqs[j], &sn, &cs);
-    sn *= magnitude;
-    cs *= magnitude;
-    T* e = x + (size_t)t * stride + (size_t)h * head_size + offset + 2 * j;
+    if (!one) angle(p, freqs[j], magnitude, sn, cs);
+    T* e = x + (size_t)h * head_size + offset + 2 * j;
     const float a = to_f32<T>(e[0]), b = to_f32<T>(e[1]);
     e[0] = from_f32<T>(a * cs - b * sn);
     e[1] = from_f32<T>(b * cs + a * sn);
   }
 }
 
-// ---- RMS norm of strided rows -----------------------------------------------------------------------
-// out[t, :] = src[t, :] * rsqrt(mean(src[t, :]^2) + eps) * w for rows that are `stride` apart (the
-// columns of one part of a wider product).
+struct EntryPlace {
+  const int* block_table;
+  int table_width, page_size, n_pages;
+  int* status;
+};
+
+// row = [R latent numbers | r key numbers]; entry = [rmsnorm(latent) * w | turned key part | zeros up to E].
+template <typename T>
+__device__ __forceinline__ void write_entry(const T* row, int slot, int p, const float* __restrict__ norm_w, float eps,
+                                            const float* __restrict__ freqs, float magnitude, T* pages,
+                                            const EntryPlace& place, int R, int r, int E, float* scratch) {
+  const int logical = p / place.page_size;
+  const int page = logical < place.table_width ? place.block_table[(size_t)slot * place.table_width + logical] : -1;
+  if (page < 0 || page >= place.n_pages) {
+    if (threadIdx.x == 0 && place.status) atomicOr(place.status, FG_STATUS_BAD_PAGE);
+    return;  // (the whole block: page is the same for every thread)
+  }
+  T* entry = pages + ((size_t)page * place.page_size + (p - logical * place.page_size)) * E;
+  norm_row<T>(row, norm_w, eps, entry, R, scratch);
+  for (int j = threadIdx.x; j < r / 2; j += blockDim.x) {
+    float sn, cs;
+    angle((float)p, freqs[j], magnitude, sn, cs);
+    const float a = to_f32<T>(row[R + 2 * j]), b = to_f32<T>(row[R + 2 * j + 1]);
+    entry[R + 2 * j] = from_f32<T>(a * cs - b * sn);
+    entry[R + 2 * j + 1] = from_f32<T>(b * cs + a * sn);
+  }
+  for (int d = R + r + threadIdx.x; d < E; d += blockDim.x) entry[d] = from_f32<T>(0.f);
+}
+
 template <typename T>
 __global__ void __launch_bounds__(128)
-rms_rows_kernel(const T* __restrict__ src, long stride, const float* __restrict__ w, float eps, T* __restrict__ out,
-                long out_stride, int dim) {
+rotate_part_kernel(T* x, long stride, const int* __restrict__ pos, const int* __restrict__ req,
+                   const float* __restrict__ freqs, float magnitude, int n_heads, int head_size, int offset,
+                   int rot_dims) {
+  const int t = blockIdx.x;
+  if (req[t] < 0) return;
+  turn_heads<T>(x + (size_t)t * stride, (float)pos[t], freqs, magnitude, n_heads, head_size, offset, rot_dims);
+}
+
+// out[t, :] = rmsnorm(src[t, :]) * w for rows that are `stride` apart (the columns of one part of a wider
+// product).
+template <typename T>
+__global__ void __launch_bounds__(128)
+rms_rows_kernel(const T* src, long stride, const float* __restrict__ w, float eps, T* out, long out_stride, int dim) {
   __shared__ float scratch[32];
-  const T* row = src + (size_t)blockIdx.x * stride;
-  float ss = 0.f;
-  for (int d = threadIdx.x; d < dim; d += blockDim.x) {
-    const float v = to_f32<T>(row[d]);
-    ss += v * v;
-  }
-  ss = block_sum(ss, scratch);
-  const float rstd = 1.f / sqrtf(ss / (float)dim + eps);
-  for (int d = threadIdx.x; d < dim; d += blockDim.x)
-    out[(size_t)blockIdx.x * out_stride + d] = from_f32<T>(to_f32<T>(row[d]) * rstd * w[d]);
+  norm_row<T>(src + (size_t)blockIdx.x * stride, w, eps, out + (size_t)blockIdx.x * out_stride, dim, scratch);
 }
 
 extern "C" int fg_rms_rows(const void* src, long stride, int dtype, const float* w, float eps, void* out,
@@ -72,45 +173,37 @@ extern "C" int fg_rms_rows(const void* src, long stride, int dtype, const float*
   return 0;
 }
 
-// ---- the cache entry -----------------------------------------------------------------------------
-// src[t] = [R latent numbers | r key numbers]; entry = [rmsnorm(latent) * w | rotated key part].
 template <typename T>
 __global__ void __launch_bounds__(128)
-latent_entry_kernel(const T* __restrict__ src, long src_stride, const float* __restrict__ norm_w, float eps,
-                    const float* __restrict__ freqs, float magnitude, T* __restrict__ pages,
-                    const int* __restrict__ block_table, int table_width, int page_size, int n_pages,
-                    const int* __restrict__ pos, const int* __restrict__ req, int R, int r, int E, int* status) {
+latent_entry_kernel(const T* src, long src_stride, const float* __restrict__ norm_w, float eps,
+                    const float* __restrict__ freqs, float magnitude, T* pages, EntryPlace place,
+                    const int* __restrict__ pos, const int* __restrict__ req, int R, int r, int E) {
   __shared__ float scratch[32];
   const int t = blockIdx.x;
   const int slot = req[t];
   if (slot < 0) return;
-  const int p = pos[t];
-  const int logical = p / page_size;
-  const int page = logical < table_width ? block_table[(size_t)slot * table_width + logical] : -1;
-  if (page < 0 || page >= n_pages) {
-    if (threadIdx.x == 0 && status) atomicOr(status, FG_STATUS_BAD_PAGE);
-    return;
-  }
-  const T* row = src + (size_t)t * src_stride;
-  T* entry = pages + ((size_t)page * page_size + (p - logical * page_size)) * E;
-  float ss = 0.f;
-  for (int d = threadIdx.x; d < R; d += blockDim.x) {
-    const float v = to_f32<T>(row[d]);
-    ss += v * v;
-  }
-  ss = block_sum(ss, scratch);
-  const float rstd = 1.f / sqrtf(ss / (float)R + eps);
-  for (int d = threadIdx.x; d < R; d += blockDim.x) entry[d] = from_f32<T>(to_f32<T>(row[d]) * rstd * norm_w[d]);
-  for (int j = threadIdx.x; j < r / 2; j += blockDim.x) {
-    float sn, cs;
-    sincosf((float)p * freqs[j], &sn, &cs);
-    sn *= magnitude;
-    cs *= magnitude;
-    const float a = to_f32<T>(row[R + 2 * j]), b = to_f32<T>(row[R + 2 * j + 1]);
-    entry[R + 2 * j] = from_f32<T>(a * cs - b * sn);
-    entry[R + 2 * j + 1] = from_f32<T>(b * cs + a * sn);
-  }
-  for (int d = R + r + threadIdx.x; d < E; d += blockDim.x) entry[d] = from_f32<T>(0.f);
+  write_entry<T>(src + (size_t)t * src_stride, slot, pos[t], norm_w, eps, freqs, magnitude, pages, place, R, r, E, scratch);
+}
+
+// blockIdx.y 0: the token's cache entry; 1: its query side, the norm of the query latent into q_out (with
+// q_norm) or the rotation of the queries' turned parts where they are.
+template <typename T>
+__global__ void __launch_bounds__(128)
+latent_prepare_kernel(const T* src, long src_stride, const float* __restrict__ norm_w, float eps,
+                      const float* __restrict__ freqs, float magnitude, T* pages, EntryPlace place,
+                      const int* __restrict__ pos, const int* __restrict__ req, int R, int r, int E, T* q, long q_stride,
+                      const float* __restrict__ q_norm, T* q_out, long q_out_stride, int q_dim, int n_heads,
+                      int head_size) {
+  __shared__ float scratch[32];
+  const int t = blockIdx.x;
+  const int slot = req[t];
+  if (slot < 0) return;
+  if (blockIdx.y == 0)
+    write_entry<T>(src + (size_t)t * src_stride, slot, pos[t], norm_w, eps, freqs, magnitude, pages, place, R, r, E, scratch);
+  else if (q_norm != nullptr)
+    norm_row<T>(q + (size_t)t * q_stride, q_norm, eps, q_out + (size_t)t * q_out_stride, q_dim, scratch);
+  else
+    turn_heads<T>(q + (size_t)t * q_stride, (float)pos[t], freqs, magnitude, n_heads, head_size, head_size - r, r);
 }
 
 // ---- attention, CUDA cores, float32 arithmetic ------------------------------------------------------
@@ -281,17 +374,46 @@ extern "C" int fg_latent_entry_write(const void* src, long src_stride, int dtype
                                      int n_tokens, int R, int r, int E, int* status, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   FG_CHECK_ARG(R > 0 && r >= 0 && r % 2 == 0 && E >= R + r, "fg_latent_entry_write: bad sizes R=%d r=%d E=%d", R, r, E);
+  const EntryPlace place{block_table, table_width, page_size, n_pages, status};
   if (dtype == FG_F32)
-    latent_entry_kernel<float><<<n_tokens, 128, 0, stream>>>((const float*)src, src_stride, norm_w, eps, freqs,
-                                                             magnitude, (float*)pages, block_table, table_width,
-                                                             page_size, n_pages, pos, req, R, r, E, status);
+    latent_entry_kernel<float><<<n_tokens, 128, 0, stream>>>((const float*)src, src_stride, norm_w, eps, freqs, magnitude,
+                                                             (float*)pages, place, pos, req, R, r, E);
   else if (dtype == FG_BF16)
-    latent_entry_kernel<__nv_bfloat16><<<n_tokens, 128, 0, stream>>>(
-        (const __nv_bfloat16*)src, src_stride, norm_w, eps, freqs, magnitude, (__nv_bfloat16*)pages, block_table,
-        table_width, page_size, n_pages, pos, req, R, r, E, status);
+    latent_entry_kernel<__nv_bfloat16><<<n_tokens, 128, 0, stream>>>((const __nv_bfloat16*)src, src_stride, norm_w, eps,
+                                                                     freqs, magnitude, (__nv_bfloat16*)pages, place, pos,
+                                                                     req, R, r, E);
   else
     FG_CHECK_ARG(false, "fg_latent_entry_write: bad dtype %d", dtype);
   FG_CHECK_LAUNCH("fg_latent_entry_write");
+  return 0;
+}
+
+// The cache entry and the query side of the step's tokens in one launch (see latent_prepare_kernel).
+// q: [n_tokens, .] rows q_stride apart; q_norm with q_out: q_dim columns are normed into q_out; without:
+// the last r numbers of each of its n_heads heads of head_size turn in place (r > 0).
+extern "C" int fg_latent_prepare(const void* src, long src_stride, int dtype, const float* norm_w, float eps,
+                                 const float* freqs, float magnitude, void* pages, const int* block_table,
+                                 int table_width, int page_size, int n_pages, const int* pos, const int* req,
+                                 int n_tokens, int R, int r, int E, void* q, long q_stride, const float* q_norm,
+                                 void* q_out, long q_out_stride, int q_dim, int n_heads, int head_size, int* status,
+                                 cudaStream_t stream) {
+  if (n_tokens == 0) return 0;
+  FG_CHECK_ARG(R > 0 && r >= 0 && r % 2 == 0 && E >= R + r, "fg_latent_prepare: bad sizes R=%d r=%d E=%d", R, r, E);
+  FG_CHECK_ARG(q_norm != nullptr ? (q_out != nullptr && q_dim > 0) : (r > 0 && r <= head_size && n_heads > 0),
+               "fg_latent_prepare: neither a query latent to norm nor heads to turn");
+  const EntryPlace place{block_table, table_width, page_size, n_pages, status};
+  const dim3 grid(n_tokens, 2);
+  if (dtype == FG_F32)
+    latent_prepare_kernel<float><<<grid, 128, 0, stream>>>(
+        (const float*)src, src_stride, norm_w, eps, freqs, magnitude, (float*)pages, place, pos, req, R, r, E, (float*)q,
+        q_stride, q_norm, (float*)q_out, q_out_stride, q_dim, n_heads, head_size);
+  else if (dtype == FG_BF16)
+    latent_prepare_kernel<__nv_bfloat16><<<grid, 128, 0, stream>>>(
+        (const __nv_bfloat16*)src, src_stride, norm_w, eps, freqs, magnitude, (__nv_bfloat16*)pages, place, pos, req, R, r,
+        E, (__nv_bfloat16*)q, q_stride, q_norm, (__nv_bfloat16*)q_out, q_out_stride, q_dim, n_heads, head_size);
+  else
+    FG_CHECK_ARG(false, "fg_latent_prepare: bad dtype %d", dtype);
+  FG_CHECK_LAUNCH("fg_latent_prepare");
   return 0;
 }
 

@@ -277,6 +277,7 @@ latent_merge_kernel(const float* __restrict__ scratch, __nv_bfloat16* __restrict
   const float f = f_s;
   for (int d = threadIdx.x; d < R; d += blockDim.x) {
     float acc = 0.f;
+#pragma unroll 8
     for (int s = 0; s < n_splits; ++s) acc = fmaf(wgt_s[s], base[(size_t)s * PART + d], acc);
     dst[d] = __float2bfloat16_rn(acc * f);
   }

@@ -13,18 +13,19 @@
 //                  with two weight stacks the result is silu(x W1^T) * (x W3^T).  This is the product of
 //                  the float32 mode and of sizes the tensor-core kernel does not take.
 //   fg_moe_gemm_mma the same product in bfloat16 on the tensor cores.
+//   fg_moe_gemm_stream the same product in bfloat16 for a few rows an expert: the experts' matrices are
+//                  streamed once (skinny_product.cuh), eight rows of the sorted list beside 16 rows of weights.
 //   fg_moe_combine ff[t, :] = sum_k weight[t, k] * y[row of (t, k), :], ascending k, and with a shared expert
 //                  that has a gate + sigmoid(gate[t]) * shared[t, :].
-#include "common.cuh"
+#include "skinny_product.cuh"
 
 // ---- the router's logits ---------------------------------------------------------------------
-// logits[t, e] = sum_k x[t, k] w[e, k] (+ bias[e]) in float32: a block of four warps a token, eight experts at a
-// time.  A thread sums runs of eight consecutive k (read as 16-byte words, all of an expert group's
+// logits[t, e] = sum_k x[t, k] w[e, k] (+ bias[e]) in float32: a block of four warps a token, eight or twelve
+// experts at a time (whichever takes fewer passes).  A thread sums runs of eight consecutive k (read as 16-byte words, all of an expert group's
 // loads in flight before the first sum: the router's matrix comes from memory at every step and a
 // chain of dependent loads would be all latency) in ascending order; the threads' sums meet in a fixed
 // exchange tree and the four warps' in ascending order, so a token's logits do not depend on the
 // batch around it.  K that is no multiple of eight, or unaligned rows, go element by element.
-constexpr int LOGITS_GROUP = 8;
 constexpr int LOGITS_THREADS = 128;
 
 template <typename T>
@@ -46,7 +47,7 @@ __device__ __forceinline__ void load8<__nv_bfloat16>(const __nv_bfloat16* p, flo
   }
 }
 
-template <typename T, bool VEC>
+template <typename T, bool VEC, int LOGITS_GROUP>
 __global__ void __launch_bounds__(LOGITS_THREADS)
 moe_logits_kernel(const T* x, long ldx, const float* __restrict__ w, long ldw, const float* __restrict__ bias,
                   float* __restrict__ logits, const int* __restrict__ req, int n_experts, int K) {
@@ -104,15 +105,19 @@ extern "C" int fg_moe_logits(const void* x, int dtype, long ldx, const float* w,
   FG_CHECK_ARG(dtype == FG_F32 || dtype == FG_BF16, "fg_moe_logits: bad dtype %d", dtype);
   const long x_words = dtype == FG_F32 ? 4 : 8;  // elements of 16 bytes
   const bool vec = K % 8 == 0 && ((uintptr_t)x & 15) == 0 && ldx % x_words == 0 && ((uintptr_t)w & 15) == 0 && ldw % 4 == 0;
+  const bool wide = (n_experts + 11) / 12 < (n_experts + 7) / 8;
 #define LAUNCH(T, VEC)                                                                                             \
-  moe_logits_kernel<T, VEC><<<n_tokens, LOGITS_THREADS, 0, stream>>>((const T*)x, ldx, w, ldw, bias, logits, req, \
+  if (wide) LAUNCH_GROUP(T, VEC, 12); else LAUNCH_GROUP(T, VEC, 8)
+#define LAUNCH_GROUP(T, VEC, G)                                                                                    \
+  moe_logits_kernel<T, VEC, G><<<n_tokens, LOGITS_THREADS, 0, stream>>>((const T*)x, ldx, w, ldw, bias, logits, req, \
                                                                      n_experts, K)
   if (dtype == FG_F32) {
-    if (vec) LAUNCH(float, true); else LAUNCH(float, false);
+    if (vec) { LAUNCH(float, true); } else { LAUNCH(float, false); }
   } else {
-    if (vec) LAUNCH(__nv_bfloat16, true); else LAUNCH(__nv_bfloat16, false);
+    if (vec) { LAUNCH(__nv_bfloat16, true); } else { LAUNCH(__nv_bfloat16, false); }
   }
 #undef LAUNCH
+#undef LAUNCH_GROUP
   FG_CHECK_LAUNCH("fg_moe_logits");
   return 0;
 }
@@ -753,6 +758,98 @@ extern "C" int fg_moe_gemm_mma(const void* x, long ldx, const void* w1, const vo
   return 0;
 }
 
+// ---- the products of a few rows an expert (bfloat16) -------------------------------------------------------
+// Tiles of up to 8 rows of one expert; a block owns 16 rows of the expert's matrix (gated: 8 gate rows and
+// the up rows of the same features) and streams them once.  A row's sums run over k in a fixed order, so
+// its value does not depend on the batch.  act (without a gate): applied to the rounded product.
+namespace {
+constexpr int STREAM_ROWS = 8;
+}
+
+template <bool GATED, int MODE>
+__global__ void __launch_bounds__(fg_skinny::THREADS)
+moe_gemm_stream_kernel(const __nv_bfloat16* x, long ldx, const __nv_bfloat16* __restrict__ w1,
+                       const __nv_bfloat16* __restrict__ w3, long w_stride, __nv_bfloat16* __restrict__ out, long ldo,
+                       int N, int K, const int* row_pair, int top, const int* tile_expert, const int* tile_row0,
+                       const int* tile_n, const int* n_tiles, int act) {
+  using namespace fg_skinny;
+  extern __shared__ __align__(16) unsigned char ring_raw[];
+  if ((int)blockIdx.y >= *n_tiles) return;
+  const int e = tile_expert[blockIdx.y], row0 = tile_row0[blockIdx.y], rows = tile_n[blockIdx.y];
+  float (*red)[ROWS][8] = reinterpret_cast<float (*)[ROWS][8]>(ring_raw);
+  BlockProduct<1, MODE> block;
+  block.begin(reinterpret_cast<uint4*>(ring_raw), K);
+  const int r = block.r, col = block.c * 8;
+  const int n0 = blockIdx.x * (GATED ? 8 : ROWS);
+  const int na = n0 + r, nb = GATED ? n0 + r : n0 + r + 8;
+  const __nv_bfloat16* wb = GATED ? w3 : w1;
+  block.row_a = na < N;
+  block.row_b = nb < N;
+  block.wa = w1 + (size_t)e * w_stride + (size_t)(block.row_a ? na : 0) * K + col;
+  block.wb = wb + (size_t)e * w_stride + (size_t)(block.row_b ? nb : 0) * K + col;
+  block.tok_ok[0] = r < rows;
+  block.first_weights();
+  int src = row0 + (r < rows ? r : 0);
+  if (row_pair != nullptr) src = row_pair[src] / top;
+  block.xr[0] = x + (size_t)src * ldx + col;
+  block.run(red);
+  if (GATED) {
+    const int i = threadIdx.x;
+    if (i >= 8 * 8) return;
+    const int tok = i / 8, f = i - tok * 8;
+    if (tok < rows && n0 + f < N) {
+      const float g = block_total<1>(red, f, tok), u = block_total<1>(red, f + 8, tok);
+      out[(size_t)(row0 + tok) * ldo + n0 + f] = __float2bfloat16_rn(g / (1.f + expf(-g)) * u);
+    }
+  } else {
+    for (int i = threadIdx.x; i < ROWS * 8; i += THREADS) {
+      const int tok = i / ROWS, row = i - tok * ROWS;
+      if (tok < rows && n0 + row < N) {
+        float v = block_total<1>(red, row, tok);
+        if (act != ACT_NONE) v = activate(__bfloat162float(__float2bfloat16_rn(v)), act);
+        out[(size_t)(row0 + tok) * ldo + n0 + row] = __float2bfloat16_rn(v);
+      }
+    }
+  }
+}
+
+extern "C" int fg_moe_stream_tile_rows() { return STREAM_ROWS; }
+
+extern "C" int fg_moe_gemm_stream(const void* x, long ldx, const void* w1, const void* w3, long w_stride, void* out,
+                                  long ldo, int N, int K, const int* row_pair, int top, const int* tile_expert,
+                                  const int* tile_row0, const int* tile_n, const int* n_tiles, int max_tiles, int act,
+                                  cudaStream_t stream) {
+  using namespace fg_skinny;
+  if (max_tiles == 0 || N == 0) return 0;
+  FG_CHECK_ARG(K > 0 && K % 8 == 0 && ldx % 8 == 0 && w_stride % 8 == 0 && max_tiles <= 65535,
+               "fg_moe_gemm_stream: bad sizes K=%d ldx=%ld tiles=%d", K, ldx, max_tiles);
+  FG_CHECK_ARG(((uintptr_t)x & 15) == 0 && ((uintptr_t)w1 & 15) == 0 && ((uintptr_t)w3 & 15) == 0,
+               "fg_moe_gemm_stream: x and the weights must be 16-byte aligned");
+  FG_CHECK_ARG(act >= ACT_NONE && act <= ACT_RELU2 && (act == ACT_NONE || w3 == nullptr),
+               "fg_moe_gemm_stream: activation %d", act);
+  typedef const __nv_bfloat16* P;
+  constexpr int MODE = THREE_AN_SM;
+  constexpr size_t smem = Ring<1, MODE>::BYTES;
+  static bool attr_set = false;
+  if (!attr_set) {
+    cudaError_t err = cudaFuncSetAttribute(moe_gemm_stream_kernel<true, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (err == cudaSuccess)
+      err = cudaFuncSetAttribute(moe_gemm_stream_kernel<false, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    FG_CHECK_ARG(err == cudaSuccess, "fg_moe_gemm_stream: shared memory: %s", cudaGetErrorString(err));
+    attr_set = true;
+  }
+  if (w3)
+    moe_gemm_stream_kernel<true, MODE><<<dim3((N + 7) / 8, max_tiles), THREADS, smem, stream>>>(
+        (P)x, ldx, (P)w1, (P)w3, w_stride, (__nv_bfloat16*)out, ldo, N, K, row_pair, top, tile_expert, tile_row0, tile_n,
+        n_tiles, act);
+  else
+    moe_gemm_stream_kernel<false, MODE><<<dim3((N + ROWS - 1) / ROWS, max_tiles), THREADS, smem, stream>>>(
+        (P)x, ldx, (P)w1, nullptr, w_stride, (__nv_bfloat16*)out, ldo, N, K, row_pair, top, tile_expert, tile_row0, tile_n,
+        n_tiles, act);
+  FG_CHECK_LAUNCH("fg_moe_gemm_stream");
+  return 0;
+}
+
 // ---- the weighted sum of a token's experts ----------------------------------------------------------
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -771,10 +868,74 @@ moe_combine_kernel(const T* y, long ldy, const float* weights, const int* pair_r
   }
 }
 
+// The same for bfloat16 rows in 16-byte pieces: a thread a piece of a token's row, the token's rows and
+// weights in shared memory, four experts' pieces in flight at a time.
+constexpr int COMBINE_THREADS = 128;
+
+__global__ void __launch_bounds__(COMBINE_THREADS)
+moe_combine_bf16x8_kernel(const __nv_bfloat16* y, long ldy, const float* weights, const int* pair_row,
+                          const __nv_bfloat16* shared, long lds, const float* gate, long ldg,
+                          __nv_bfloat16* __restrict__ out, long ldo, int dim, int top) {
+  extern __shared__ int rows_s[];  // [top] rows, then [top] weights
+  float* w_s = reinterpret_cast<float*>(rows_s + top);
+  const int t = blockIdx.x, piece = blockIdx.y * COMBINE_THREADS + threadIdx.x;
+  for (int k = threadIdx.x; k < top; k += COMBINE_THREADS) {
+    rows_s[k] = pair_row[(size_t)t * top + k];
+    w_s[k] = weights[(size_t)t * top + k];
+  }
+  const bool in = piece * 8 < dim;
+  uint4 s4 = make_uint4(0u, 0u, 0u, 0u);
+  float g = 1.f;
+  if (shared != nullptr && in) {
+    s4 = *reinterpret_cast<const uint4*>(shared + (size_t)t * lds + piece * 8);
+    if (gate != nullptr) g = 1.f / (1.f + expf(-gate[(size_t)t * ldg]));
+  }
+  __syncthreads();
+  if (!in) return;
+  float acc[8];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) acc[i] = 0.f;
+  auto add = [&](const uint4& raw, float w) {
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 f = __bfloat1622float2(h[i]);
+      acc[2 * i] = fmaf(w, f.x, acc[2 * i]);
+      acc[2 * i + 1] = fmaf(w, f.y, acc[2 * i + 1]);
+    }
+  };
+  for (int k0 = 0; k0 < top; k0 += 4) {
+    uint4 raw[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int r = k0 + j < top ? rows_s[k0 + j] : -1;
+      raw[j] = r >= 0 ? *reinterpret_cast<const uint4*>(y + (size_t)r * ldy + piece * 8) : make_uint4(0u, 0u, 0u, 0u);
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+      if (k0 + j < top && rows_s[k0 + j] >= 0) add(raw[j], w_s[k0 + j]);
+  }
+  if (shared != nullptr) add(s4, g);
+  uint4 o4;
+  __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&o4);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) o2[i] = __floats2bfloat162_rn(acc[2 * i], acc[2 * i + 1]);
+  *reinterpret_cast<uint4*>(out + (size_t)t * ldo + piece * 8) = o4;
+}
+
 // shared: [n_tokens, dim] or null (added, times sigmoid(gate[t * ldg]) with a gate)
 extern "C" int fg_moe_combine(const void* y, long ldy, const float* weights, const int* pair_row, const void* shared,
                               long lds, const float* gate, long ldg, void* out, long ldo, int dtype, int n_tokens, int dim, int top, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
+  const auto ok16 = [](const void* p, long ld) { return ((uintptr_t)p & 15) == 0 && ld % 8 == 0; };
+  if (dtype == FG_BF16 && dim % 8 == 0 && top <= 1024 && ok16(y, ldy) && ok16(out, ldo) && ok16(shared, lds)) {
+    const dim3 grid(n_tokens, (dim / 8 + COMBINE_THREADS - 1) / COMBINE_THREADS);
+    moe_combine_bf16x8_kernel<<<grid, COMBINE_THREADS, (size_t)top * 8, stream>>>(
+        (const __nv_bfloat16*)y, ldy, weights, pair_row, (const __nv_bfloat16*)shared, lds, gate, ldg, (__nv_bfloat16*)out,
+        ldo, dim, top);
+    FG_CHECK_LAUNCH("fg_moe_combine");
+    return 0;
+  }
   if (dtype == FG_F32)
     moe_combine_kernel<float><<<n_tokens, 256, 0, stream>>>((const float*)y, ldy, weights, pair_row, (const float*)shared, lds,
                                                             gate, ldg, (float*)out, ldo, dim, top);

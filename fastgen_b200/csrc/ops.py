@@ -39,6 +39,8 @@ def _ptr(t: Optional[torch.Tensor]):
 
 
 _P, _I, _F = c_void_p, c_int, c_float
+#: most (token, expert) pairs whose products stream the experts' matrices (tiles of eight rows)
+MOE_STREAM_PAIRS = 64
 #: (token, expert) pairs from which the experts' products go to the vendor's grouped product
 MOE_GROUPED_PAIRS = 512
 _L = ctypes.c_long
@@ -54,6 +56,8 @@ _CORE_SIGNATURES = {
     "fg_gated_part_norm": [_P, _L, _P, _L, _I, _P, _P, _L, _P, _I, _I, _I, _F, _P],
     "fg_rms_rows": [_P, _L, _I, _P, _F, _P, _L, _I, _I, _P],
     "fg_rotate_part": [_P, _L, _I, _P, _P, _P, _F, _I, _I, _I, _I, _I, _P],
+    "fg_latent_prepare": [_P, _L, _I, _P, _F, _P, _F, _P, _P, _I, _I, _I, _P, _P, _I, _I, _I, _I, _P, _L, _P, _P, _L, _I, _I, _I,
+                          _P, _P],
     "fg_latent_entry_write": [_P, _L, _I, _P, _F, _P, _F, _P, _P, _I, _I, _I, _P, _P, _I, _I, _I, _I, _P, _P],
     "fg_latent_attention_simt": [_P, _I, _L, _L, _P, _L, _L, _P, _L, _L, _I, _P, _L, _P, _P, _I, _I, _I, _P, _P, _P,
                                  _P, _I, _I, _I, _I, _I, _F, _P, _P],
@@ -198,6 +202,7 @@ _MOE_SIGNATURES = {
     "fg_moe_gather": [_P, _L, _P, _L, _I, _P, _P, _I, _I, _I, _I, _P],
     "fg_moe_gemm": [_P, _L, _P, _P, _L, _P, _L, _I, _I, _I, _P, _I, _P, _P, _P, _P, _I, _P],
     "fg_moe_gemm_mma": [_P, _L, _P, _P, _L, _P, _L, _I, _I, _P, _I, _P, _P, _P, _P, _I, _P],
+    "fg_moe_gemm_stream": [_P, _L, _P, _P, _L, _P, _L, _I, _I, _P, _I, _P, _P, _P, _P, _I, _I, _P],
     "fg_moe_combine": [_P, _L, _P, _P, _P, _L, _P, _L, _P, _L, _I, _I, _I, _I, _P],
 }
 _RECUR_SIGNATURES = {
@@ -501,6 +506,29 @@ class Ops:
             _ptr(ctx.pos), _ptr(ctx.req), src.shape[0], rank, rot_dim, pages.shape[-1], _ptr(self.status),
             _stream()))
 
+    def latent_prepare(self, src, norm_weight, eps: float, freqs, magnitude: float, memory, ctx, rank: int, rot_dim: int,
+                       q, q_norm=None, n_heads: int = 0, head_size: int = 0) -> torch.Tensor:
+        """``latent_entry_write`` and the query side in one launch: with ``q_norm`` the result is
+        ``rms_rows(q, q_norm, eps)`` (rows of padding tokens are left unwritten), without it the last
+        ``rot_dim`` numbers of each of the ``n_heads`` heads of ``q`` are turned in place (``rotate_part``)
+        and ``q`` is the result."""
+        pages = memory.k_pages
+        assert src.stride(1) == 1 and src.shape[1] == rank + rot_dim and pages.is_contiguous()
+        assert norm_weight.dtype == torch.float32 and norm_weight.numel() == rank
+        assert q.stride(1) == 1 and q.dtype == src.dtype and q.shape[0] == src.shape[0]
+        out = q
+        if q_norm is not None:
+            assert q_norm.dtype == torch.float32 and q_norm.numel() == q.shape[1]
+            out = torch.empty(q.shape, dtype=q.dtype, device=q.device)
+        else:
+            assert q.shape[1] == n_heads * head_size
+        _check(self.lib, self.lib.fg_latent_prepare(
+            _ptr(src), src.stride(0), _code(src.dtype), _ptr(norm_weight), float(eps), _ptr(freqs), float(magnitude),
+            _ptr(pages), _ptr(memory.block_table), memory.block_table.shape[1], memory.page_size, pages.shape[0],
+            _ptr(ctx.pos), _ptr(ctx.req), src.shape[0], rank, rot_dim, pages.shape[-1], _ptr(q), q.stride(0), _ptr(q_norm),
+            _ptr(out), out.stride(0), q.shape[1], n_heads, head_size, _ptr(self.status), _stream()))
+        return out
+
     def latent_attention(self, qa, qt, out, gate, memory, ctx, n_heads: int, rank: int, rot_dim: int,
                          scale: float) -> torch.Tensor:
         """Causal softmax attention of ``n_heads`` query heads on the one cached entry per token:
@@ -774,7 +802,8 @@ class Ops:
         """``sum_k weights[t, k] * expert_{ids[t, k]}(x[t])`` with expert ``e`` the gated feed-forward
         ``w2[e] (silu(w1[e] x) * (w3[e] x))``; ``w1``, ``w3`` [E, F, K] (each expert's matrix contiguous,
         the experts a fixed stride apart: they may be the halves of ``w13`` [E, 2F, K]) and ``w2``
-        [E, K, F].  The (token, choice) pairs are sorted by expert on the device.  Few pairs: the
+        [E, K, F].  The (token, choice) pairs are sorted by expert on the device.  A few pairs in
+        bfloat16 (single tokens): the chosen experts' matrices are streamed once.  Some more: the
         products run over tiles of one expert's rows, on the tensor cores in bfloat16 where the sizes
         allow, else (and in float32) with float32 sums in ascending order.  Many pairs in bfloat16 (a
         prompt portion), given ``w13``: the sorted rows are gathered and the two products are the
@@ -802,7 +831,9 @@ class Ops:
         mma = (not grouped and x.dtype == torch.bfloat16 and k % 8 == 0 and f % 8 == 0 and x.stride(0) % 8 == 0
                and w_stride % 8 == 0 and x.data_ptr() % 16 == 0 and w1.data_ptr() % 16 == 0
                and (not gated or w3.data_ptr() % 16 == 0) and hasattr(lib, "fg_moe_gemm_mma") and not os.environ.get("FG_NO_MOE_MMA"))
-        tile_rows = lib.fg_moe_mma_tile_rows() if mma else lib.fg_moe_gemm_tile_rows()
+        stream = mma and pairs <= MOE_STREAM_PAIRS and w2.data_ptr() % 16 == 0
+        tile_rows = (lib.fg_moe_stream_tile_rows() if stream else lib.fg_moe_mma_tile_rows() if mma
+                     else lib.fg_moe_gemm_tile_rows())
         max_tiles = -(-pairs // tile_rows) + n_experts - 1
         plan = torch.empty(2 * pairs + 3 * max_tiles + 1 + n_experts, dtype=torch.int32, device=x.device)
         row_pair, pair_row = plan[:pairs], plan[pairs : 2 * pairs]
@@ -831,7 +862,14 @@ class Ops:
             mid = (torch.empty if gated else torch.zeros)((pairs, f), dtype=x.dtype, device=x.device)
             y = torch.empty((pairs, k), dtype=x.dtype, device=x.device)
             tiles = (_ptr(tile_expert), _ptr(tile_row0), _ptr(tile_n), _ptr(n_tiles), max_tiles, _stream())
-            if mma:
+            if stream:
+                # a few rows an expert: the matrices are streamed once, the activation is an epilogue
+                _check(lib, lib.fg_moe_gemm_stream(_ptr(x), x.stride(0), _ptr(w1), _ptr(w3), w_stride, _ptr(mid),
+                                                   mid.stride(0), f, k, _ptr(row_pair), top, *tiles[:-1],
+                                                   0 if gated else ACTIVATIONS[act], tiles[-1]))
+                _check(lib, lib.fg_moe_gemm_stream(_ptr(mid), mid.stride(0), _ptr(w2), None, w2.stride(0), _ptr(y),
+                                                   y.stride(0), k, f, None, top, *tiles[:-1], 0, tiles[-1]))
+            elif mma:
                 _check(lib, lib.fg_moe_gemm_mma(_ptr(x), x.stride(0), _ptr(w1), _ptr(w3), w_stride, _ptr(mid),
                                                 mid.stride(0), f, k, _ptr(row_pair), top, *tiles))
                 if not gated:

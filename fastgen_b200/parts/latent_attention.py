@@ -115,15 +115,25 @@ class LatentAttention(Mixer):
         t, H, R = x.shape[0], p.n_heads, p.kv_rank
         down = ops.linear(x, self.w_down)
         gate = down[:, self.gate_offset : self.gate_offset + self.gate_size] if p.gate else None
-        if memory.writes:
-            ops.latent_entry_write(down[:, self.entry_offset : self.entry_offset + R + p.rot_dim], self.dkv_norm, p.eps, self.freqs,
-                                   self.magnitude, memory, ctx, R, p.rot_dim)
-        if p.q_rank is None:
-            q = down[:, : H * self.qk]
+        turn = (ctx, self.freqs, self.magnitude, H, self.qk, p.head_dim, p.rot_dim)
+        q = down[:, : p.q_rank if p.q_rank is not None else H * self.qk]
+        if memory.writes and (p.q_rank is not None or p.rot_dim):
+            # the cache entries and what the queries need first, in one launch
+            q = ops.latent_prepare(down[:, self.entry_offset : self.entry_offset + R + p.rot_dim], self.dkv_norm, p.eps,
+                                   self.freqs, self.magnitude, memory, ctx, R, p.rot_dim, q,
+                                   q_norm=self.dq_norm if p.q_rank is not None else None, n_heads=H, head_size=self.qk)
         else:
-            q = ops.linear(ops.rms_rows(down[:, : p.q_rank], self.dq_norm, p.eps), self.w_uq)
-        if p.rot_dim:
-            ops.rotate_part(q, ctx, self.freqs, self.magnitude, H, self.qk, p.head_dim, p.rot_dim)
+            if memory.writes:
+                ops.latent_entry_write(down[:, self.entry_offset : self.entry_offset + R + p.rot_dim], self.dkv_norm,
+                                       p.eps, self.freqs, self.magnitude, memory, ctx, R, p.rot_dim)
+            if p.q_rank is not None:
+                q = ops.rms_rows(q, self.dq_norm, p.eps)
+            elif p.rot_dim:
+                ops.rotate_part(q, *turn)
+        if p.q_rank is not None:
+            q = ops.linear(q, self.w_uq)
+            if p.rot_dim:
+                ops.rotate_part(q, *turn)
         q = q.view(t, H, self.qk)
         # the key map folded into the queries: qa[h] = q_plain[h] @ w_uk[h]
         qa = ops.head_products(q[:, :, : p.head_dim], self.w_uk, self.w_uk_t)  # [H, T, R]

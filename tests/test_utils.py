@@ -59,7 +59,7 @@ def test_every_declared_signature_belongs_to_its_library():
     int_only = {"fg_attention_decode_scratch_floats", "fg_attention_decode_split", "fg_attention_prefill_rows",
                 "fg_attention_rows_per_block", "fg_last_error", "fg_attention_sigmoid_decode_keys",
                 "fg_latent_mma_rows", "fg_latent_mma_keys", "fg_latent_mma_scratch_floats",
-                "fg_moe_gemm_tile_rows", "fg_moe_mma_tile_rows", "fg_mlstm_state_floats"}
+                "fg_moe_gemm_tile_rows", "fg_moe_mma_tile_rows", "fg_moe_stream_tile_rows", "fg_mlstm_state_floats"}
     assert undeclared <= int_only, undeclared - int_only
 
 
