@@ -55,6 +55,8 @@ CORE_SOURCES = [
     "selftest.cu",
 ]
 
+LATENT_SOURCES = ["latent_mma.cu", "latent_tcgen05.cu", "errors.cu"]
+
 _loaded: Dict[str, ctypes.CDLL] = {}
 _lock = threading.Lock()
 
@@ -220,7 +222,7 @@ def moe_library() -> ctypes.CDLL:
 
 def latent_library(rank: int, rot_dim: int) -> ctypes.CDLL:
     """The tensor-core kernels of the attention over a cached latent, compiled per latent size."""
-    return load(f"fg_latent_r{rank}_t{rot_dim}", ["latent_mma.cu", "errors.cu"],
+    return load(f"fg_latent_r{rank}_t{rot_dim}", LATENT_SOURCES,
                 [f"FG_LATENT_RANK={rank}", f"FG_LATENT_ROT={rot_dim}"])
 
 
@@ -231,7 +233,7 @@ def latent_mma_supported(rank: int, rot_dim: int) -> bool:
         and -(-(rank + rot_dim) // 16) * 16 <= 640
 
 
-def build_all(head_dims: Sequence[int] = (16, 32, 64, 128), latent_sizes: Sequence = ((512, 64), (256, 32))) -> None:
+def build_all(head_dims: Sequence[int] = (16, 32, 64, 128), latent_sizes: Sequence = ((512, 64), (256, 32), (512, 0), (256, 0))) -> None:
     """Compile every library (used by the build check and before shipping); the latent-attention
     library for the given (latent, rotated part) sizes."""
     _compile("fg_core", CORE_SOURCES)
@@ -239,7 +241,7 @@ def build_all(head_dims: Sequence[int] = (16, 32, 64, 128), latent_sizes: Sequen
     _compile("fg_moe", ["moe.cu", "errors.cu"])
     _compile("fg_recur", ["mlstm.cu", "rglru.cu", "errors.cu"])
     for rank, rot in latent_sizes:
-        _compile(f"fg_latent_r{rank}_t{rot}", ["latent_mma.cu", "errors.cu"],
+        _compile(f"fg_latent_r{rank}_t{rot}", LATENT_SOURCES,
                  [f"FG_LATENT_RANK={rank}", f"FG_LATENT_ROT={rot}"])
     for hd in head_dims:
         _compile(f"fg_attn_hd{hd}", ["attention.cu", "errors.cu"], [f"FG_HEAD_DIM={hd}"])

@@ -39,6 +39,9 @@ def _ptr(t: Optional[torch.Tensor]):
 
 
 _P, _I, _F = c_void_p, c_int, c_float
+#: fewest blocks of a launch of the latent attention's tcgen05 kernel (fewer: the mma.sync kernel, which
+#: cuts a tile's keys into stretches)
+LATENT_TC5_BLOCKS = 32
 #: most (token, expert) pairs whose products stream the experts' matrices (tiles of eight rows)
 MOE_STREAM_PAIRS = 64
 #: (token, expert) pairs from which the experts' products go to the vendor's grouped product
@@ -173,6 +176,8 @@ _latent = {}
 _LATENT_SIGNATURES = {
     "fg_latent_attention_mma": [_P, _L, _L, _P, _L, _L, _P, _L, _L, _P, _L, _P, _P, _I, _I, _I, _P, _P, _P, _P, _I, _I,
                                 _I, _I, _I, _F, _I, _I, _P, ctypes.c_longlong, _P, _P],
+    "fg_latent_attention_tc5": [_P, _P, _L, _L, _P, _L, _L, _P, _L, _L, _P, _L, _P, _I, _I, _I, _P, _P, _P, _P, _I, _I, _I,
+                                _I, _I, _F, _P, _P],
 }
 
 
@@ -329,6 +334,7 @@ class Ops:
         # captured graphs may hold their addresses
         self._split = {}
         self._split_retired = []
+        self._latent_maps = {}  # (address, shape, box) of a layer's latent pool -> its tensor map
         self.use_tcgen05 = not bool(os.environ.get("FG_NO_TCGEN05"))
         # library products accumulate and reduce in float32 (no bfloat16 split-K sums)
         torch.backends.cuda.matmul.allow_bf16_reduced_precision_reduction = False
@@ -544,8 +550,11 @@ class Ops:
         even = all(v % 2 == 0 for v in (*qa.stride()[:2], *qt.stride()[:2], *out.stride()[:2], qt.storage_offset()))
         if (qa.dtype == torch.bfloat16 and out.dtype == torch.bfloat16 and even
                 and build.latent_mma_supported(rank, rot_dim) and pages.shape[-1] == -(-(rank + rot_dim) // 8) * 8):
-            # bfloat16: the tensor cores; few tiles (single tokens) are cut into stretches of keys
+            # bfloat16: the tensor cores.  Prompt portions of some size: the tcgen05 kernel.  Few tiles
+            # (single tokens): mma.sync, the keys cut into stretches
             lib = latent(rank, rot_dim)
+            if self._latent_tc5(lib, qa, qt, out, gate, memory, ctx, n_heads, rank, rot_dim, scale):
+                return out
             rows, keys = lib.fg_latent_mma_rows(), lib.fg_latent_mma_keys()
             tiles = ctx.attention_tiles(attention_tiling(n_heads, 1, rows), 1)
             max_keys = tiles.max_keys or memory.block_table.shape[1] * memory.page_size
@@ -576,6 +585,35 @@ class Ops:
             _ptr(ctx.pos), _ptr(tiles.req), _ptr(tiles.tok0), _ptr(tiles.ntok), tiles.n, n_heads, rank, rot_dim,
             pages.shape[-1], float(scale), _ptr(self.status), _stream()))
         return out
+
+    def _latent_tc5(self, lib, qa, qt, out, gate, memory, ctx, n_heads: int, rank: int, rot_dim: int, scale: float) -> bool:
+        """``latent_attention`` on the tcgen05 kernel; ``False`` where it does not apply: latent sizes it is
+        not built for, pages that are no power of two, strides of no 16 bytes, steps that are mostly
+        single tokens, and launches of a few blocks."""
+        rows, page = lib.fg_latent_tc5_rows(), memory.page_size
+        if not rows or not self.use_tcgen05 or page < 8 or page & (page - 1) or ctx.n_tokens < 4 * ctx.n_seqs:
+            return False
+        if any(v % 8 for v in (*qa.stride()[:2], *out.stride()[:2])) or qa.data_ptr() % 16 or out.data_ptr() % 16:
+            return False
+        per_tile = attention_tiling(n_heads, 1, rows)
+        blocks = -(-ctx.n_tokens // per_tile) * -(-n_heads // min(n_heads, rows)) * lib.fg_latent_tc5_blocks_a_tile()
+        if blocks < LATENT_TC5_BLOCKS:
+            return False
+        tiles = ctx.attention_tiles(per_tile, 1)
+        pages = memory.k_pages
+        box = min(page, lib.fg_latent_tc5_keys())
+        key = (pages.data_ptr(), pages.shape[0], page, pages.shape[-1], box)
+        tm = self._latent_maps.get(key)
+        if tm is None:
+            tm = self._latent_maps[key] = TensorMap()
+            _check(self.lib, self.lib.fg_make_kv_tensor_map(tm.ptr, _ptr(pages), 1, pages.shape[0], 1, page, pages.shape[-1], box))
+            Ops.launches -= 1  # not a kernel
+        _check(lib, lib.fg_latent_attention_tc5(
+            tm.ptr, _ptr(qa), qa.stride(1), qa.stride(0), _ptr(qt), qt.stride(0), qt.stride(1), _ptr(out), out.stride(1),
+            out.stride(0), _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(memory.block_table),
+            memory.block_table.shape[1], page, pages.shape[0], _ptr(ctx.pos), _ptr(tiles.req), _ptr(tiles.tok0),
+            _ptr(tiles.ntok), tiles.n, n_heads, rank, rot_dim, pages.shape[-1], float(scale), _ptr(self.status), _stream()))
+        return True
 
     def embedding_bigram(self, table, bigram, tokens, pos, req, last_token, out, buckets: int, mul_prev: int,
                          mul_cur: int) -> torch.Tensor:

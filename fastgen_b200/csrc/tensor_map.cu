@@ -31,7 +31,9 @@ PFN_cuTensorMapEncodeTiled_v12000 encoder() {
 extern "C" int fg_make_kv_tensor_map(void* out_map, const void* base, int n_layers, int n_pages,
                                      int n_kv_heads, int page_size, int head_dim, int box_rows) {
   FG_CHECK_ARG(((uintptr_t)out_map & 63) == 0, "fg_make_kv_tensor_map: the map must be 64-byte aligned");
-  FG_CHECK_ARG(head_dim % 64 == 0, "fg_make_kv_tensor_map: head size %d is not a multiple of 64", head_dim);
+  // (rows are 16-byte multiples; columns of a box beyond the row's end are filled with zeros)
+  FG_CHECK_ARG(head_dim % 8 == 0 && head_dim >= 64, "fg_make_kv_tensor_map: head size %d is not a multiple of 8 from 64 on",
+               head_dim);
   FG_CHECK_ARG(box_rows > 0 && box_rows <= 256 && box_rows <= page_size,
                "fg_make_kv_tensor_map: bad box of %d rows for pages of %d", box_rows, page_size);
   auto encode = encoder();

@@ -65,7 +65,7 @@ class _Shape:
                         ("seq_slot", max_seqs), ("seq_start", max_seqs + 1), ("seq_cached", max_seqs)):
             self.off[name] = self.size
             self.size += n
-        self.capacity = self.size + 3 * 4 * (n_tokens + max_seqs + 8) + 4  # room for four tile lists
+        self.capacity = self.size + 12 * (3 * (n_tokens + max_seqs) + 1)  # room for twelve tile lists
         self.dev = torch.zeros(self.capacity, dtype=torch.int32, device=device)
         self.ring = [torch.zeros(self.capacity, dtype=torch.int32).pin_memory() for _ in range(_RING)]
         self.ring_events: List[Optional[torch.cuda.Event]] = [None] * _RING

@@ -42,7 +42,7 @@ def test_every_declared_signature_belongs_to_its_library():
         return names
     core = exported(build.CORE_SOURCES)
     attn = exported(["attention.cu"])
-    latent = exported(["latent_mma.cu"])
+    latent = exported(["latent_mma.cu", "latent_tcgen05.cu"])
     delta = exported(["delta_rule.cu"])
     moe = exported(["moe.cu"])
     recur = exported(["mlstm.cu", "rglru.cu"])
@@ -58,6 +58,7 @@ def test_every_declared_signature_belongs_to_its_library():
     undeclared -= set(ops._DELTA_SIGNATURES) | set(ops._MOE_SIGNATURES) | set(ops._RECUR_SIGNATURES)
     int_only = {"fg_attention_decode_scratch_floats", "fg_attention_decode_split", "fg_attention_prefill_rows",
                 "fg_attention_rows_per_block", "fg_last_error", "fg_attention_sigmoid_decode_keys",
+                "fg_latent_tc5_rows", "fg_latent_tc5_keys", "fg_latent_tc5_blocks_a_tile",
                 "fg_latent_mma_rows", "fg_latent_mma_keys", "fg_latent_mma_scratch_floats",
                 "fg_moe_gemm_tile_rows", "fg_moe_mma_tile_rows", "fg_moe_stream_tile_rows", "fg_mlstm_state_floats"}
     assert undeclared <= int_only, undeclared - int_only
