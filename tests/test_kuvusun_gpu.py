@@ -529,6 +529,67 @@ def test_keys_at_page_and_tile_borders(dtype, mode):
 
 
 @pytest.mark.gpu
+@pytest.mark.parametrize("page", [8, 64, 256])
+@pytest.mark.parametrize("sizes", [(4, 64, 0), (6, 64, 16), (32, 256, 32), (3, 256, 0), (24, 128, 10), (5, 192, 6), (24, 512, 64),
+                                   (8, 512, 0), (130, 256, 64), (1, 64, 4), (7, 384, 40)])
+def test_prompt_kernel_on_tensor_memory(monkeypatch, sizes, page):
+    """The tcgen05 kernel of prompt portions by itself, at once and on cached entries, with and without a
+    gate per head, for latents of one and of two output halves, tiles of 64 and of 32 keys, more heads
+    than a block has rows, turned parts that fill no group of columns and start at no 16 bytes; against
+    float64 sums over the same bfloat16 entries.  A loud key sits on every border of a tile or page, and
+    the pages' free places hold large numbers that no query may see."""
+    from fastgen_b200.cache import CacheManager
+    from fastgen_b200.csrc import ops as ops_module
+    from fastgen_b200.parts import CacheSpec
+
+    heads, rank, rot = sizes
+    monkeypatch.setattr(ops_module, "LATENT_TC5_BLOCKS", 1)
+    ops = _ops(torch.bfloat16)
+    lib = ops_module.latent(rank, rot)
+    assert lib.fg_latent_tc5_rows() == 128
+    g = torch.Generator().manual_seed(heads + rank + rot)
+    width = -(-(rank + rot) // 8) * 8
+    total = 210
+    cache = CacheManager([CacheSpec(1, width, None, n_pools=1)], [None], [None], page, -(-total // page) + 2, 2, 2 * total,
+                         dtype=torch.bfloat16, device=DEV, tensor_map_factory=ops.make_kv_tensor_maps)
+    req = cache.admit("r")
+    cache.reserve(req, total)
+    cache.flush_tables()
+    mem = cache.memory(0)
+    entries = torch.randn(total, width, generator=g).bfloat16()
+    for j in (0, 31, 32, 63, 64, 127, 128, 191, 192):
+        entries[j, :rank] *= 2
+    entries[:, rank + rot :] = 0
+    mem.k_pages[:] = 1000.0
+    table = mem.block_table[req.slot].tolist()
+    for j in range(total):
+        mem.k_pages[table[j // page], 0, j % page] = entries[j].to(DEV)
+    scale = 2.0 / (rank + rot) ** 0.5
+    keys = entries.double()
+    for start, n, gated in ((0, 210, False), (77, 133, True), (190, 20, False)):
+        qa = torch.randn(heads, n, rank, generator=g).bfloat16()
+        q = torch.randn(n, heads, rot + 6, generator=g).bfloat16().to(DEV)
+        gate = torch.randn(n, heads, generator=g).bfloat16()
+        out = torch.full((heads, n, rank), float("nan"), dtype=torch.bfloat16, device=DEV)
+        launched = ops_module.Ops.launches
+        assert ops._latent_tc5(lib, qa.to(DEV), q[:, :, 6:] if rot else qa.to(DEV).permute(1, 0, 2), out,
+                               gate.to(DEV) if gated else None, mem, _context(req.slot, start, n), heads, rank, rot, scale)
+        assert ops_module.Ops.launches == launched + 1
+        ops.check_status()
+        s = torch.einsum("hnd,kd->hnk", qa.double(), keys[:, :rank])
+        if rot:
+            s = s + torch.einsum("nhd,kd->hnk", q[:, :, 6:].double().cpu(), keys[:, rank : rank + rot])
+        later = torch.arange(total)[None, :] > torch.arange(start, start + n)[:, None]
+        ref = torch.softmax((s * scale).masked_fill(later[None], float("-inf")), dim=-1) @ keys[:, :rank]
+        if gated:
+            ref = ref * torch.sigmoid(gate.double()).T[:, :, None]
+        _close(out.double().cpu(), ref, torch.bfloat16)
+        # (a row's own rounding, not the largest row's)
+        err = (out.double().cpu() - ref).norm(dim=-1) / ref.norm(dim=-1)
+        assert float(err.max()) < 0.01, float(err.max())
+
+
+@pytest.mark.gpu
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 def test_a_reader_uses_the_other_layers_entries(dtype):
     """A mixer without a latent projection reads the entries that another one wrote, with its own heads,
@@ -839,6 +900,34 @@ def test_many_live_requests(tmp_path, dtype):
     steps = H.plan_many(requests, seed=4, max_live=12)
     outputs, engine = H.run_engine(d, dtype, steps, 16, H.max_live_tokens(steps, 16) + 32, max_requests=12)
     compare(d, requests, H.collect(steps, outputs), dtype)
+
+
+@pytest.mark.gpu
+def test_portions_on_either_side_of_the_prompt_kernels_threshold(tmp_path):
+    """A model whose latents the tcgen05 kernel takes, in bfloat16: long portions run there, short ones and
+    single tokens on the kernel that cuts a tile's keys into stretches, all on the same cached entries."""
+    from fastgen_b200.csrc.ops import Ops
+
+    cfg = dict(architecture="Kuvusun", vocab=150, width=120, norm=dict(eps=1e-5, groups=2), layers=[
+        _layer(_turned(40, 16, 16, 8, 64, 0.2, 3000.0), _dense(72)), _layer(_plain(33, 16, 8, 40, 128, 0.2), _dense(64)),
+        _layer(_turned(20, 8, 16, 16, 64, 0.25, 3000.0, kv_from=0), None)])
+    d = write_random_model(Path(tmp_path) / "m", cfg, 4, dtype=torch.bfloat16, norm_jitter=0.3, std=0.1)
+    taken = []
+    inner = Ops._latent_tc5
+
+    def spy(self, *args):
+        taken.append(inner(self, *args))
+        return taken[-1]
+    requests = _requests(150, [260, 170], 21)
+    try:
+        Ops._latent_tc5 = spy
+        for sizes in ((260,), (150, 1, 1, 2, 3, 103), (17, 130, 1, 9, 103)):
+            steps = H.plan_portions(requests, sizes=sizes)
+            outputs, _ = H.run_engine(d, torch.bfloat16, steps, 16, H.max_live_tokens(steps, 16) + 32)
+            compare(d, requests, H.collect(steps, outputs), torch.bfloat16)
+    finally:
+        Ops._latent_tc5 = inner
+    assert any(taken) and not all(taken)
 
 
 @pytest.mark.gpu
