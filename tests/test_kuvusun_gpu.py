@@ -530,7 +530,7 @@ def test_keys_at_page_and_tile_borders(dtype, mode):
 
 @pytest.mark.gpu
 @pytest.mark.parametrize("page", [8, 64, 256])
-@pytest.mark.parametrize("sizes", [(4, 64, 0), (6, 64, 16), (32, 256, 32), (3, 256, 0), (24, 128, 10), (5, 192, 6), (24, 512, 64),
+@pytest.mark.parametrize("sizes", [(5, 64, 0), (7, 64, 24), (32, 256, 32), (3, 256, 0), (24, 128, 10), (5, 192, 6), (24, 512, 64),
                                    (8, 512, 0), (130, 256, 64), (1, 64, 4), (7, 384, 40)])
 def test_prompt_kernel_on_tensor_memory(monkeypatch, sizes, page):
     """The tcgen05 kernel of prompt portions by itself, at once and on cached entries, with and without a
