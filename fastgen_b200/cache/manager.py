@@ -8,7 +8,7 @@ fastgen/cache.py:37-140) is generalised here:
 * runs of layers whose mixers need the same thing per token (head count, head
   size, window) form a *group*; each group has a page pool of its own, storage
   of its own and a block table of its own per request;
-* a group with a window gives pages back as soon as the window has passed them;
+* a group with a window (or with chunks) gives pages back as soon as no later query sees them;
 * every live request holds one *slot*: the row of its block tables on the
   device and the index of its fixed-size state (zeroed on admission), for
   mixers that keep state of fixed size instead of per-token entries.
@@ -94,7 +94,9 @@ class CacheGroup:
     dirty: List[Tuple[int, int, int]] = field(default_factory=list)  # (slot, col, page)
 
     def first_needed_page(self, length: int) -> int:
-        """Lowest logical page of the window of a query at position >= ``length``."""
+        """Lowest logical page that a query at position >= ``length`` sees (apart from kept ones)."""
+        if self.spec.chunk is not None:
+            return length // self.spec.chunk * self.spec.chunk // self.page_size
         if self.spec.window is None:
             return 0
         return max(0, length - self.spec.window + 1) // self.page_size
@@ -349,7 +351,7 @@ class CacheManager:
 
     def advance(self, req: RequestCache, new_length: int) -> None:
         """Record that ``req`` now holds ``new_length`` tokens and give back the
-        pages a window has passed."""
+        pages a window or a chunk has passed."""
         if new_length < req.length:
             raise CacheError("a request's length cannot shrink")
         req.length = new_length
@@ -361,7 +363,7 @@ class CacheManager:
                 for lp in gone:
                     grp.host_table[req.slot, lp] = -1
                     grp.dirty.append((req.slot, lp, -1))
-                # a window shorter than a page can leave a group without a page behind the kept ones
+                # a window shorter than a page, or a chunk that has ended, can leave a group without a page behind the kept ones
                 # at a page's edge: the bound shrinks to what the remaining pages cover, and the
                 # next reservation looks at the maps
                 held = req.pages[gi]

@@ -18,6 +18,7 @@ from . import zeladra as _zeladra  # registers Zeladra
 from . import tanupel as _tanupel  # registers Tanupel
 from . import palulorn as _palulorn  # registers Palulorn
 from . import kuvusun as _kuvusun  # registers Kuvusun
+from . import pegurax as _pegurax  # registers Pegurax
 
 __all__ = [
     "ConfigError",

@@ -13,7 +13,7 @@
 //    positions [128 s, 128 s + 128), whatever else is in the batch.
 //
 // Semantics as in attention_simt.cuh (fastgen/forward.py:176-258): scores
-// q.k * scale over positions j <= pos (and j > pos - window), softmax and the
+// q.k * scale over positions j <= pos (and j > pos - window, or those of the query's chunk), softmax and the
 // running maximum / sum / output in float32 (exp2f on log2e-scaled scores),
 // probabilities rounded to bfloat16 for the second product, as the tensor core
 // needs.  Keys and values are read from pages laid out [page, kv_head, slot, HD].
@@ -284,8 +284,8 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv
     cp_async_wait<0>();
     return;
   }
-  const int k_lo = window > 0 ? max(0, min_pos - window + 1) / PREFILL_KEYS * PREFILL_KEYS : 0;
-  const int k_begin = window > 0 ? max(0, min_pos - window + 1) : 0;
+  const int k_begin = first_visible(min_pos, window);
+  const int k_lo = k_begin / PREFILL_KEYS * PREFILL_KEYS;
   const int k_end = max_pos + 1;
   const int* table_row = block_table + (size_t)b * table_width;
   // tiles of kept first positions that lie wholly before the window's first tile
@@ -314,6 +314,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv
   // the warp's 16 rows; this thread's two rows
   const int r0 = warp * 16 + (lane >> 2), r1 = r0 + 8;
   const int p0 = row_pos[r0], p1 = row_pos[r1];
+  const int lo0 = first_visible(p0, window), lo1 = first_visible(p1, window);
   int warp_max = -1;
   for (int r = warp * 16; r < warp * 16 + 16; ++r) warp_max = max(warp_max, row_pos[r]);
 
@@ -372,7 +373,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv
         for (int e = 0; e < 4; ++e) {
           const int j = k0 + nt * 8 + 2 * (lane & 3) + (e & 1);
           const int p = (e < 2) ? p0 : p1;
-          const bool vis = p >= 0 && j <= p && (window <= 0 || j > p - window || j < keep_first);
+          const bool vis = p >= 0 && j <= p && (j >= (e < 2 ? lo0 : lo1) || j < keep_first);
           if (SIGMOID) {
             float wgt;
             {
@@ -507,7 +508,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
   const int p = pos[tok];
   const int k0 = split * DECODE_SPLIT;
   if (k0 > p) return;  // this split lies beyond the request's keys
-  const int k_begin = window > 0 ? max(0, p - window + 1) : 0;
+  const int k_begin = first_visible(p, window);
   if (window <= 0) keep_first = 0;
   if (k0 + DECODE_SPLIT <= k_begin && k0 >= keep_first) return;  // wholly before the window, nothing kept
   const int k_end = p + 1;
@@ -661,7 +662,7 @@ attention_combine_kernel(const float* scratch, __nv_bfloat16* __restrict__ out, 
   // a padding lane has no request: nothing is written for it (its token index may be any row,
   // also one that belongs to a request of the step)
   if (request < 0) return;
-  const int s_lo = window > 0 ? max(0, p - window + 1) / DECODE_SPLIT : 0;
+  const int s_lo = first_visible(p, window) / DECODE_SPLIT;
   int s_hi = p / DECODE_SPLIT;  // inclusive
   if (s_hi >= max_splits) {
     // the launch was sized for shorter requests: report instead of reading past the scratch

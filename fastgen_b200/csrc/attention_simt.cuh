@@ -11,7 +11,8 @@
 //
 // Semantics of fastgen/forward.py:176-258: softmax(q.k * scale) v over the
 // positions j <= pos(query) of the query's own request (and, when a window is given,
-// j > pos - window or j < keep_first: the first positions stay visible), grouped-query heads h -> h / (Hq/Hkv).
+// j > pos - window or j < keep_first: the first positions stay visible; with a negative window only the
+// positions of the query's own chunk, see first_visible), grouped-query heads h -> h / (Hq/Hkv).
 // Running maximum, sum and output accumulator are float32; exp is expf.  With `sinks` (float32 per
 // query head) the denominator also holds exp(sink_h): a score without a key, unscaled, counted once.
 //
@@ -90,18 +91,21 @@ attention_simt_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ out
   if (max_pos < 0) return;
   // with a window, tiles that lie wholly before the earliest row's window are skipped, apart
   // from those that hold some of the first `keep_first` positions, which stay visible for good
+  const int lo_min = first_visible(min_pos, window);
   int k_win = 0, k_keep_end = 0;
-  if (window > 0) {
-    k_win = max(0, min_pos - window + 1) / KEYS * KEYS;
+  if (window != 0) {
+    k_win = lo_min / KEYS * KEYS;
     k_keep_end = min(k_win, (max(keep_first, 0) + KEYS - 1) / KEYS * KEYS);
   }
 
   // this thread's 4 score rows: warp, warp+4, warp+8, warp+12; column = lane
   float m_run[4], l_run[4];
+  int row_lo[4];  // the first position each of them sees
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
     m_run[i] = -INFINITY;
     l_run[i] = 0.f;
+    row_lo[i] = first_visible(row_pos[warp + 4 * i], window);
     // a sink: a learned score per query head that has no key and no value and counts once in the
     // denominator; the running maximum and sum start from it
     if (sinks != nullptr && row_head(warp + 4 * i) < group) {
@@ -126,7 +130,7 @@ attention_simt_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ out
         const int page = logical < table_width ? block_table[(size_t)b * table_width + logical] : -1;
         if (page >= 0 && page < n_pages) {
           base = (((long long)page * n_kv_heads + g) * page_size + (j - logical * page_size)) * HD;
-        } else if (window <= 0 || j > min_pos - window || j < keep_first) {
+        } else if (j >= lo_min || j < keep_first) {
           // a key some row must see has no page
           if (status) atomicOr(status, FG_STATUS_BAD_PAGE);
         }
@@ -160,7 +164,7 @@ attention_simt_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ out
     for (int i = 0; i < 4; ++i) {
       const int r = warp + 4 * i;
       const int p = row_pos[r];
-      const bool visible = has_key && p >= 0 && j <= p && (window <= 0 || j > p - window || j < keep_first);
+      const bool visible = has_key && p >= 0 && j <= p && (j >= row_lo[i] || j < keep_first);
       // with a cap, the scaled score is squashed to cap * tanh(score / cap)
       float sc = s[i] * scale;
       if (softcap > 0.f) sc = softcap * tanhf(sc / softcap);

@@ -333,7 +333,7 @@ attention_prefill_tc5_kernel(const __grid_constant__ CUtensorMap k_map, const __
       if (!SPLIT) stage_queries();
       const int min_pos = SPLIT ? pos[tok0] : first_pos_s;  // tokens of a tile are consecutive positions
       const int max_pos = min_pos + ntok - 1;
-      const int k_begin = window > 0 ? max(0, min_pos - window + 1) : 0;
+      const int k_begin = first_visible(min_pos, window);
       const int k_end = max_pos + 1;
       const int item_tiles = (k_end - k_begin / KEYS * KEYS + KEYS - 1) / KEYS;
       // this part's key tiles: the item's are cut into stretches of equal length, at most `parts`
@@ -522,6 +522,8 @@ attention_prefill_tc5_kernel(const __grid_constant__ CUtensorMap k_map, const __
           warp_max = max(warp_max, __shfl_xor_sync(0xffffffffu, warp_max, o));
           warp_min = min(warp_min, __shfl_xor_sync(0xffffffffu, warp_min, o));
         }
+        // the first position this row sees, and the first one from which every row of the warp sees keys
+        const int my_lo = first_visible(my_pos, window), warp_lo = first_visible(warp_max, window);
         for (int t = 0; t < n_tiles; ++t) {
           const int gt = base + t, stage = gt & 1;
           const uint32_t s_addr = tmem + my_lane + COL_S0 + stage * KEYS;
@@ -536,7 +538,7 @@ attention_prefill_tc5_kernel(const __grid_constant__ CUtensorMap k_map, const __
             for (int i = 0; i < KEYS; ++i) s[i] = fmaf(-2.f, rcp_approx(1.f + ex2_approx(s[i] * two_l2e)), 1.f);
           }
           const bool need_mask =
-              !warp_full || k0 + KEYS - 1 > warp_min || (window > 0 && k0 <= warp_max - window);
+              !warp_full || k0 + KEYS - 1 > warp_min || k0 < warp_lo;
           float alpha = 1.f;
           bool raise = false;
           float sum = 0.f;
@@ -562,7 +564,7 @@ attention_prefill_tc5_kernel(const __grid_constant__ CUtensorMap k_map, const __
                 // (the weight first, then the choice: computed only where visible, the chain of special
                 // functions ran behind a branch: 126 us instead of 80 at head size 128)
                 const float wgt = weight(sv, i);
-                const bool vis = !need_mask || (my_pos >= 0 && j <= my_pos && (window <= 0 || j > my_pos - window));
+                const bool vis = !need_mask || (my_pos >= 0 && j <= my_pos && j >= my_lo);
                 return vis ? wgt : 0.f;
               };
 #pragma unroll
@@ -573,7 +575,7 @@ attention_prefill_tc5_kernel(const __grid_constant__ CUtensorMap k_map, const __
 #pragma unroll
             for (int i = 0; i < KEYS; ++i) {
               const int j = k0 + i;
-              const bool vis = my_pos >= 0 && j <= my_pos && (window <= 0 || j > my_pos - window);
+              const bool vis = my_pos >= 0 && j <= my_pos && j >= my_lo;
               if (!vis) s[i] = -INFINITY;
             }
           }

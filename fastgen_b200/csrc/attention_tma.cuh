@@ -126,7 +126,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __g
   const int p = pos[tok];
   const int k0 = split * SPLIT;
   if (k0 > p) return;
-  const int k_begin = window > 0 ? max(0, p - window + 1) : 0;
+  const int k_begin = first_visible(p, window);
   if (k0 + SPLIT <= k_begin) return;
   const int k_end = p + 1;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -342,7 +342,7 @@ attention_decode_persistent_kernel(const __grid_constant__ CUtensorMap k_map,
   // are the (request, split, kv head) triples that exist, numbered request by request, so
   // that block b takes items b, b + G, ... and every block gets the same number of them.
   // Positions are inputs of the step (no kernel of the step writes them).
-  auto first_split = [&](int p) { return window > 0 ? max(0, p - window + 1) / SPLIT : 0; };
+  auto first_split = [&](int p) { return first_visible(p, window) / SPLIT; };
   for (int sq = tid; sq < n_seqs; sq += PS_THREADS) s_pos[sq] = seq_req[sq] < 0 ? -1 : pos[seq_tok[sq]];
   __syncthreads();
   if (warp == 0) {
@@ -399,7 +399,7 @@ attention_decode_persistent_kernel(const __grid_constant__ CUtensorMap k_map,
     seq = lo;
     p = s_pos[seq];
     split = first_split(p) + (r - s_cum[seq]);
-    k_begin = window > 0 ? max(0, p - window + 1) : 0;
+    k_begin = first_visible(p, window);
     return true;
   };
 
@@ -720,7 +720,7 @@ attention_prefill_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __
   // tokens of a tile are consecutive positions: the extremes are at its ends
   const int min_pos = row_pos[0];
   const int max_pos = min_pos + ntok - 1;
-  const int k_begin = window > 0 ? max(0, min_pos - window + 1) : 0;
+  const int k_begin = first_visible(min_pos, window);
   const int k_lo = k_begin / PF_KEYS * PF_KEYS;
   const int k_end = max_pos + 1;
   // with a window, the sequence's first keep_first positions stay visible: the key tiles that
@@ -795,6 +795,7 @@ attention_prefill_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __
 
   const int r0 = warp * 16 + (lane >> 2), r1 = r0 + 8;
   const int p0 = row_pos[r0], p1 = row_pos[r1];
+  const int lo0 = first_visible(p0, window), lo1 = first_visible(p1, window);
   int warp_max = -1, warp_min = 0x7fffffff;
   bool warp_full = true;  // all 16 rows of the warp hold a query
   for (int r = warp * 16; r < warp * 16 + 16; ++r) {
@@ -802,6 +803,7 @@ attention_prefill_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __
     warp_max = max(warp_max, p);
     if (p >= 0) warp_min = min(warp_min, p); else warp_full = false;
   }
+  const int warp_lo = first_visible(warp_max, window);  // from here on every row of the warp sees keys
   uint32_t qf[HD / 16][4];
 #pragma unroll
   for (int kk = 0; kk < HD / 16; ++kk)
@@ -834,7 +836,7 @@ attention_prefill_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __
       qk_product_swz<HD, NT, PF_HALF>(s, qf, ks, 0, lane);
       // only tiles that touch the diagonal, the window's edge or an unused row need the mask
       const bool need_mask = !warp_full || k0 + PF_KEYS - 1 > warp_min || t < n_keep ||
-                             (window > 0 && k0 <= warp_max - window);
+                             k0 < warp_lo;
       if (need_mask) {
 #pragma unroll
         for (int nt = 0; nt < NT; ++nt)
@@ -842,7 +844,7 @@ attention_prefill_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __
           for (int e = 0; e < 4; ++e) {
             const int j = k0 + nt * 8 + 2 * (lane & 3) + (e & 1);
             const int p = (e < 2) ? p0 : p1;
-            const bool vis = p >= 0 && j <= p && (window <= 0 || j > p - window || j < keep_first);
+            const bool vis = p >= 0 && j <= p && (j >= (e < 2 ? lo0 : lo1) || j < keep_first);
             if (!vis) s[nt][e] = -INFINITY;
           }
       }

@@ -43,6 +43,8 @@ CORE_SOURCES = [
     "part_norm.cu",
     "dyt.cu",
     "stream_norm.cu",
+    "layer_norm_pair.cu",
+    "selective_scan.cu",
     "mamba2.cu",
     "latent.cu",
     "activation.cu",

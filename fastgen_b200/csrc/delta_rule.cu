@@ -13,7 +13,8 @@
 //   qn, kn [T, kv heads, DP]; rec [T, heads, DP + 4] = the decay's DP numbers, beta, k . q, 0, 0;
 //   vp [T, heads, DVP]        (DP: d rounded up to the kernel's row count, DVP: dv up to a multiple of 4)
 // The second runs the recurrence, which is a chain from token to token whose length, not the
-// arithmetic, sets the time, so nothing else is left in it.  A block of eight warps works on
+// arithmetic, sets the time, so nothing else is left in it (with one decay per head instead of one per
+// channel, `rec` holds g, beta, k . q, 0 and the decay is one number a token).  A block of eight warps works on
 // (sequence, head, a run of the state's columns).  A column's rows are spread over LPC lanes, RPL
 // rows a lane in registers (in runs of four: a lane reads its part of k, g and q as 16-byte words);
 // a warp holds 32 / LPC columns and the sums over a column's rows end in log2(LPC) exchanges.
@@ -33,7 +34,8 @@ constexpr int DELTA_MAX_NRP = 8;  // key sizes up to 256
 
 __device__ __forceinline__ float softplus_f32(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 
-template <typename TA>
+// HEAD: a is [T, heads] and dt_bias [heads], one decay per head
+template <typename TA, bool HEAD>
 __global__ void __launch_bounds__(128)
 delta_prepare_kernel(const float* qkv, long qkv_stride, const TA* a, long a_stride, const TA* b, long b_stride,
                      const float* __restrict__ dt_bias, const float* __restrict__ a_log, const int* __restrict__ req,
@@ -62,7 +64,8 @@ delta_prepare_kernel(const float* qkv, long qkv_stride, const TA* a, long a_stri
   ssk = warp_sum(ssk);
   const float rq = (1.f / sqrtf((float)d)) / sqrtf(ssq + 1e-6f), rk = 1.f / sqrtf(ssk + 1e-6f);
   const float rate = expf(a_log[h]);
-  float* rec_row = rec + ((size_t)t * n_heads + h) * (DP + 4);
+  const int REC = HEAD ? 4 : DP + 4;
+  float* rec_row = rec + ((size_t)t * n_heads + h) * REC;
   const bool first = h == hk * group;  // the group's first head writes the group's q and k
   float* qn_row = qn + ((size_t)t * n_kv_heads + hk) * DP;
   float* kn_row = kn + ((size_t)t * n_kv_heads + hk) * DP;
@@ -78,13 +81,19 @@ delta_prepare_kernel(const float* qkv, long qkv_stride, const TA* a, long a_stri
         kn_row[r] = kv;
       }
       // rows beyond d: k and q are zero there, and so is the state
-      rec_row[r] = r < d ? expf(-rate * softplus_f32(to_f32<TA>(a[(size_t)t * a_stride + h * d + r]) + dt_bias[h * d + r])) : 0.f;
+      if (!HEAD)
+        rec_row[r] = r < d ? expf(-rate * softplus_f32(to_f32<TA>(a[(size_t)t * a_stride + h * d + r]) + dt_bias[h * d + r])) : 0.f;
     }
   }
   kq = warp_sum(kq);
   if (lane < 4) {
     const float beta = 1.f / (1.f + expf(-to_f32<TA>(b[(size_t)t * b_stride + h])));
-    rec_row[DP + lane] = lane == 0 ? beta : (lane == 1 ? kq : 0.f);
+    if (HEAD) {
+      const float g = expf(-rate * softplus_f32(to_f32<TA>(a[(size_t)t * a_stride + h]) + dt_bias[h]));
+      rec_row[lane] = lane == 0 ? g : (lane == 1 ? beta : (lane == 2 ? kq : 0.f));
+    } else {
+      rec_row[DP + lane] = lane == 0 ? beta : (lane == 1 ? kq : 0.f);
+    }
   }
   float* vp_row = vp + ((size_t)t * n_heads + h) * DVP;
   for (int c = lane; c < DVP; c += 32) vp_row[c] = c < dv ? row[v_off + c] : 0.f;
@@ -96,7 +105,7 @@ __device__ __forceinline__ void delta_copy16(float* dst, const float* src, bool 
                "r"(bytes) : "memory");
 }
 
-template <int LPC, int RPL>
+template <int LPC, int RPL, bool HEAD>
 __global__ void __launch_bounds__(DELTA_THREADS)
 delta_scan_kernel(const float* __restrict__ qn, const float* __restrict__ kn, const float* __restrict__ rec,
                   const float* __restrict__ vp, float* __restrict__ out, long out_stride, float* __restrict__ state,
@@ -105,11 +114,11 @@ delta_scan_kernel(const float* __restrict__ qn, const float* __restrict__ kn, co
   constexpr int DP = LPC * RPL;            // rows, padded
   constexpr int CPW = 32 / LPC;            // columns a warp
   constexpr int COLS = DELTA_WARPS * CPW;  // columns a block
-  constexpr int REC = DP + 4;
+  constexpr int REC = HEAD ? 4 : DP + 4;
   static_assert(DP % 32 == 0 && RPL % 4 == 0 && COLS % 4 == 0, "rows in runs of four, a multiple of 32 in all");
   extern __shared__ __align__(16) float smem[];
-  // per token of a buffer: q[DP], k[DP], rec[DP + 4] (g, beta, k . q), v[COLS]
-  constexpr int TOKF = 3 * DP + 4 + COLS;
+  // per token of a buffer: q[DP], k[DP], rec (g, beta, k . q), v[COLS]
+  constexpr int TOKF = 2 * DP + REC + COLS;
   constexpr int BUF = DELTA_TOKENS * TOKF;
   constexpr int CHUNKS = TOKF / 4;  // 16-byte words a token
   const int slot = seq_slot[blockIdx.z];
@@ -161,12 +170,14 @@ delta_scan_kernel(const float* __restrict__ qn, const float* __restrict__ kn, co
     const float4* sq = reinterpret_cast<const float4*>(tokp);
     const float4* sk = reinterpret_cast<const float4*>(tokp + DP);
     const float4* sg = reinterpret_cast<const float4*>(tokp + 2 * DP);
-    const float beta = tokp[3 * DP], kq = tokp[3 * DP + 1], v = tokp[3 * DP + 4 + cw];
+    constexpr int AT = HEAD ? 2 * DP + 1 : 3 * DP;  // beta's place
+    const float beta = tokp[AT], kq = tokp[AT + 1], v = tokp[2 * DP + REC + cw];
+    const float g_head = HEAD ? tokp[2 * DP] : 0.f;
     float kr[RPL];
     float rk2[4] = {0.f, 0.f, 0.f, 0.f}, rq2[4] = {0.f, 0.f, 0.f, 0.f};  // four chains a sum: a lane's rows are many
 #pragma unroll
     for (int jj = 0; jj < RPL / 4; ++jj) {
-      const float4 kv = sk[sub + LPC * jj], gv = sg[sub + LPC * jj], qv = sq[sub + LPC * jj];
+      const float4 kv = sk[sub + LPC * jj], gv = HEAD ? make_float4(g_head, g_head, g_head, g_head) : sg[sub + LPC * jj], qv = sq[sub + LPC * jj];
       const float ke[4] = {kv.x, kv.y, kv.z, kv.w}, ge[4] = {gv.x, gv.y, gv.z, gv.w}, qe[4] = {qv.x, qv.y, qv.z, qv.w};
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
@@ -225,14 +236,15 @@ delta_scan_kernel(const float* __restrict__ qn, const float* __restrict__ kn, co
 // rows of the prepared arrays for key size d (the row count of the kernel that takes it)
 static int delta_rows(int d) { return d <= 32 ? 32 : d <= 64 ? 64 : d <= 128 ? 128 : 256; }
 
+template <bool HEAD>
 static int launch_scan(cudaStream_t stream, const float* qn, const float* kn, const float* rec, const float* vp,
                        float* out, long out_stride, float* state, long state_stride, const int* seq_slot,
                        const int* seq_start, int n_seqs, int n_heads, int n_kv_heads, int d, int dv, int DVP) {
 #define CASE(LPC, RPL)                                                                                         \
   {                                                                                                            \
     constexpr int COLS = DELTA_WARPS * (32 / LPC);                                                             \
-    const size_t smem = (size_t)DELTA_STAGES * DELTA_TOKENS * (3 * LPC * RPL + 4 + COLS) * sizeof(float);       \
-    auto kern = delta_scan_kernel<LPC, RPL>;                                                                    \
+    const size_t smem = (size_t)DELTA_STAGES * DELTA_TOKENS * ((HEAD ? 2 : 3) * LPC * RPL + 4 + COLS) * sizeof(float); \
+    auto kern = delta_scan_kernel<LPC, RPL, HEAD>;                                                              \
     if (smem > 48 * 1024) {                                                                                     \
       cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);       \
       FG_CHECK_ARG(e == cudaSuccess, "fg_delta_scan: shared memory: %s", cudaGetErrorString(e));                \
@@ -256,14 +268,14 @@ extern "C" long fg_delta_scan_scratch_floats(int n_tokens, int n_heads, int n_kv
 }
 
 // qkv: float32 [T, q (kv heads x d) | k (kv heads x d) | v (heads x dv)], the convolutions' outputs.
-// a: [T, heads x d] decay logits and b: [T, .] step-size logits (column h of row t at b[t * b_stride + h]),
-// both of `dtype`.  dt_bias: float32 [heads x d]; a_log: float32 [heads].  out: float32 [T, heads x dv].
+// a: [T, heads x d] decay logits ([T, heads] with head_decay: one decay per head) and b: [T, .] step-size logits (column h of row t at b[t * b_stride + h]),
+// both of `dtype`.  dt_bias: float32 [heads x d] or [heads]; a_log: float32 [heads].  out: float32 [T, heads x dv].
 // state: float32 [slots, state_stride], a slot's first heads * dv * d numbers.
 extern "C" int fg_delta_scan(const float* qkv, long qkv_stride, const void* a, long a_stride, const void* b,
                              long b_stride, int dtype, const float* dt_bias, const float* a_log, float* out,
                              long out_stride, float* state, long state_stride, const int* seq_slot,
                              const int* seq_start, int n_seqs, const int* req, int n_tokens, float* scratch,
-                             int n_heads, int n_kv_heads, int d, int dv, cudaStream_t stream) {
+                             int n_heads, int n_kv_heads, int d, int dv, int head_decay, cudaStream_t stream) {
   if (n_seqs == 0 || n_tokens == 0) return 0;
   FG_CHECK_ARG(n_heads > 0 && n_kv_heads > 0 && n_heads % n_kv_heads == 0, "fg_delta_scan: %d heads over %d key heads",
                n_heads, n_kv_heads);
@@ -274,34 +286,37 @@ extern "C" int fg_delta_scan(const float* qkv, long qkv_stride, const void* a, l
   float* qn = scratch;
   float* kn = qn + (size_t)n_tokens * n_kv_heads * DP;
   float* rec = kn + (size_t)n_tokens * n_kv_heads * DP;
-  float* vp = rec + (size_t)n_tokens * n_heads * (DP + 4);
+  float* vp = rec + (size_t)n_tokens * n_heads * (head_decay ? 4 : DP + 4);
   const int blocks = (int)(((long)n_tokens * n_heads + 3) / 4);
-  if (dtype == FG_F32)
-    delta_prepare_kernel<float><<<blocks, 128, 0, stream>>>(qkv, qkv_stride, (const float*)a, a_stride, (const float*)b,
-                                                            b_stride, dt_bias, a_log, req, qn, kn, rec, vp, n_tokens,
-                                                            n_heads, n_kv_heads, d, dv, DP, DVP);
-  else if (dtype == FG_BF16)
-    delta_prepare_kernel<__nv_bfloat16><<<blocks, 128, 0, stream>>>(
-        qkv, qkv_stride, (const __nv_bfloat16*)a, a_stride, (const __nv_bfloat16*)b, b_stride, dt_bias, a_log, req, qn,
-        kn, rec, vp, n_tokens, n_heads, n_kv_heads, d, dv, DP, DVP);
-  else
-    FG_CHECK_ARG(false, "fg_delta_scan: bad dtype %d", dtype);
+  FG_CHECK_ARG(dtype == FG_F32 || dtype == FG_BF16, "fg_delta_scan: bad dtype %d", dtype);
+#define PREPARE(T, HEAD)                                                                                        \
+  delta_prepare_kernel<T, HEAD><<<blocks, 128, 0, stream>>>(qkv, qkv_stride, (const T*)a, a_stride, (const T*)b,  \
+                                                            b_stride, dt_bias, a_log, req, qn, kn, rec, vp,       \
+                                                            n_tokens, n_heads, n_kv_heads, d, dv, DP, DVP)
+  if (dtype == FG_F32) {
+    if (head_decay) PREPARE(float, true); else PREPARE(float, false);
+  } else {
+    if (head_decay) PREPARE(__nv_bfloat16, true); else PREPARE(__nv_bfloat16, false);
+  }
+#undef PREPARE
   FG_CHECK_LAUNCH("fg_delta_scan (prepare)");
-  const int rc = launch_scan(stream, qn, kn, rec, vp, out, out_stride, state, state_stride, seq_slot, seq_start, n_seqs,
-                             n_heads, n_kv_heads, d, dv, DVP);
+  const auto scan = head_decay ? launch_scan<true> : launch_scan<false>;
+  const int rc = scan(stream, qn, kn, rec, vp, out, out_stride, state, state_stride, seq_slot, seq_start, n_seqs,
+                      n_heads, n_kv_heads, d, dv, DVP);
   if (rc != 0) return rc;
   FG_CHECK_LAUNCH("fg_delta_scan");
   return 0;
 }
 
 // ---- the read-out's norm and gate -------------------------------------------------------------
-// out[t, h, :] = o[t, h, :] * rsqrt(mean(o[t, h, :]^2) + eps) * w[:] * sigmoid(z[t, h, :]); a warp a
+// out[t, h, :] = o[t, h, :] * rsqrt(mean(o[t, h, :]^2) + eps) * w[:] * sigmoid(z[t, h, :]), or silu(z) with
+// `silu`; a warp a
 // (token, head), float32 arithmetic, one rounding.
 template <typename TZ>
 __global__ void __launch_bounds__(128)
 head_norm_gate_kernel(const float* o, long o_stride, const TZ* z, long z_stride, const float* __restrict__ w,
                       TZ* __restrict__ out, long out_stride, const int* __restrict__ req, int n_tokens, int n_heads,
-                      int dv, float eps) {
+                      int dv, float eps, int silu) {
   const int item = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (item >= n_tokens * n_heads) return;
   const int t = item / n_heads, h = item - t * n_heads;
@@ -312,23 +327,24 @@ head_norm_gate_kernel(const float* o, long o_stride, const TZ* z, long z_stride,
   ss = warp_sum(ss);
   const float rstd = rsqrtf(ss / (float)dv + eps);
   for (int c = lane; c < dv; c += 32) {
-    const float gate = 1.f / (1.f + expf(-to_f32<TZ>(z[(size_t)t * z_stride + h * dv + c])));
+    const float zc = to_f32<TZ>(z[(size_t)t * z_stride + h * dv + c]);
+    const float gate = (silu ? zc : 1.f) / (1.f + expf(-zc));
     out[(size_t)t * out_stride + h * dv + c] = from_f32<TZ>(src[c] * rstd * w[c] * gate);
   }
 }
 
 extern "C" int fg_head_norm_gate(const float* o, long o_stride, const void* z, long z_stride, int dtype,
                                  const float* w, void* out, long out_stride, const int* req, int n_tokens,
-                                 int n_heads, int dv, float eps, cudaStream_t stream) {
+                                 int n_heads, int dv, float eps, int silu, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   const int blocks = (n_tokens * n_heads + 3) / 4;
   if (dtype == FG_F32)
     head_norm_gate_kernel<float><<<blocks, 128, 0, stream>>>(o, o_stride, (const float*)z, z_stride, w, (float*)out,
-                                                             out_stride, req, n_tokens, n_heads, dv, eps);
+                                                             out_stride, req, n_tokens, n_heads, dv, eps, silu);
   else if (dtype == FG_BF16)
     head_norm_gate_kernel<__nv_bfloat16><<<blocks, 128, 0, stream>>>(o, o_stride, (const __nv_bfloat16*)z, z_stride, w,
                                                                      (__nv_bfloat16*)out, out_stride, req, n_tokens,
-                                                                     n_heads, dv, eps);
+                                                                     n_heads, dv, eps, silu);
   else
     FG_CHECK_ARG(false, "fg_head_norm_gate: bad dtype %d", dtype);
   FG_CHECK_LAUNCH("fg_head_norm_gate");

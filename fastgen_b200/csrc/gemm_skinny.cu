@@ -16,7 +16,7 @@
 // Two fused variants serve the decode step:
 //  * epilogue "SwiGLU": W holds gate and up rows interleaved in blocks of 8 (rows
 //    16b..16b+7 gate, 16b+8..16b+15 up of features 8b..8b+7), so a block's 16 rows
-//    are gate and up of the same 8 features and it writes silu(gate) * up
+//    are gate and up of the same 8 features and it writes silu(gate) * up (or relu(gate) * up)
 //    (fastgen/forward.py:491-495) -- the [gate | up] intermediate never exists;
 //  * epilogue "QKV": the 16 output rows are 8 adjacent pairs of one head; they are
 //    rotated by the token's position (fastgen/kernels/rope.py:77-89), queries go
@@ -34,7 +34,7 @@ using namespace fg_skinny;
 enum { EPI_PLAIN = 0, EPI_QKV = 1, EPI_SWIGLU = 2 };
 
 // What the epilogues may need beyond the sums: a bias over the output rows (all epilogues) and
-// an activation (plain epilogue), and for the fused query/key/value projection the positions,
+// an activation (plain epilogue; SwiGLU epilogue: 1 for a relu gate), and for the fused query/key/value projection the positions,
 // tables and pages.
 struct QkvEpilogue {
   const __nv_bfloat16* bias;  // [N] or null
@@ -68,14 +68,14 @@ __device__ __forceinline__ void epilogue_plain(float (*red)[ROWS][NT * 8], TO* y
 
 // rows 0..7 are the gates and rows 8..15 the ups of features n0/2 .. n0/2+7
 template <int NT, typename TO>
-__device__ __forceinline__ void epilogue_swiglu(float (*red)[ROWS][NT * 8], TO* y, int ldy, int M, int N, int n0) {
+__device__ __forceinline__ void epilogue_swiglu(float (*red)[ROWS][NT * 8], TO* y, int ldy, int M, int N, int n0, int relu) {
   for (int i = threadIdx.x; i < 8 * NT * 8; i += THREADS) {
     const int tok = i / 8, f = i - tok * 8;
     if (tok < M && n0 + 8 + f < N) {
       const float g = block_total<NT>(red, f, tok), u = block_total<NT>(red, f + 8, tok);
       // both are rounded to bfloat16 first, as a separate gate kernel would see them
       const float gr = __bfloat162float(__float2bfloat16_rn(g)), ur = __bfloat162float(__float2bfloat16_rn(u));
-      y[(size_t)tok * ldy + n0 / 2 + f] = from_f32<TO>(gr / (1.f + expf(-gr)) * ur);
+      y[(size_t)tok * ldy + n0 / 2 + f] = from_f32<TO>((relu ? fmaxf(gr, 0.f) : gr / (1.f + expf(-gr))) * ur);
     }
   }
 }
@@ -134,7 +134,7 @@ gemm_skinny_kernel(const __nv_bfloat16* x, int ldx, const __nv_bfloat16* __restr
   if (EPI == EPI_PLAIN) {
     epilogue_plain<NT, TO>(red, y, ldy, M, N, n0, qkv.bias, qkv.act);
   } else if (EPI == EPI_SWIGLU) {
-    epilogue_swiglu<NT, TO>(red, y, ldy, M, N, n0);
+    epilogue_swiglu<NT, TO>(red, y, ldy, M, N, n0, qkv.act);
   } else {
     // the block's 16 rows are 8 adjacent pairs of one head of q, k or v; a thread's pair,
     // angle and destination were worked out before the main loop
@@ -238,14 +238,15 @@ extern "C" int fg_gemm_skinny_bf16(const void* x, int ldx, const void* w, int ld
   return 0;
 }
 
-// y[M, F] = silu(x W1^T) * (x W3^T) for w = W1 and W3 interleaved in blocks of 8 rows
+// y[M, F] = silu(x W1^T) * (x W3^T) (relu instead of silu with `relu`) for w = W1 and W3 interleaved in blocks of 8 rows
 // ([2F, K]: rows 16b..16b+7 are rows 8b..8b+7 of W1, rows 16b+8..16b+15 those of W3).
 extern "C" int fg_gemm_skinny_swiglu_bf16(const void* x, int ldx, const void* w, int ldw, void* y, int ldy,
-                                          int M, int F, int K, cudaStream_t stream) {
+                                          int M, int F, int K, int relu, cudaStream_t stream) {
   if (M == 0 || F == 0) return 0;
   FG_CHECK_ARG(F % 8 == 0, "fg_gemm_skinny_swiglu_bf16: the feed-forward width %d is not a multiple of 8", F);
   if (check_common("fg_gemm_skinny_swiglu_bf16", x, ldx, w, ldw, ldy, M, F, K, K)) return -1;
   QkvEpilogue none{};
+  none.act = relu;
   launch<__nv_bfloat16, EPI_SWIGLU>(x, ldx, w, ldw, y, ldy, M, 2 * F, K, none, stream);
   FG_CHECK_LAUNCH("fg_gemm_skinny_swiglu_bf16");
   return 0;

@@ -15,8 +15,10 @@
 //   fg_moe_gemm_mma the same product in bfloat16 on the tensor cores.
 //   fg_moe_gemm_stream the same product in bfloat16 for a few rows an expert: the experts' matrices are
 //                  streamed once (skinny_product.cuh), eight rows of the sorted list beside 16 rows of weights.
+//                  All three take `in_w` (null: ones), the router's weights, where a weight multiplies the
+//                  expert's input instead of its output: a row's sums are multiplied by its pair's weight.
 //   fg_moe_combine ff[t, :] = sum_k weight[t, k] * y[row of (t, k), :], ascending k, and with a shared expert
-//                  that has a gate + sigmoid(gate[t]) * shared[t, :].
+//                  that has a gate + sigmoid(gate[t]) * shared[t, :].  Null weights stand for ones.
 #include "skinny_product.cuh"
 
 // ---- the router's logits ---------------------------------------------------------------------
@@ -269,7 +271,10 @@ moe_route_groups_kernel(const float* logits, long ldl, const float* __restrict__
 #pragma unroll
   for (int i = 0; i < ROUTE_MAX_PER_LANE; ++i) {
     const int e = lane + 32 * i;
-    c[i] = e < n_experts ? s[i] + (correction ? correction[e] : 0.f) : -INFINITY;
+    // (sigmoid scores without a correction and without groups: the logits rank, scores may round to equal)
+    const float rank = correction ? s[i] + correction[min(e, n_experts - 1)]
+                                  : (kind == 1 && n_groups == 0 && e < n_experts ? logits[(size_t)t * ldl + e] : s[i]);
+    c[i] = e < n_experts ? rank : -INFINITY;
     if (e < n_experts) s_s[w][e] = s[i];
   }
   if (n_groups > 0) {
@@ -501,7 +506,8 @@ template <typename T, bool GATED>
 __global__ void __launch_bounds__(256)
 moe_gemm_kernel(const T* x, long ldx, const T* __restrict__ w1, const T* __restrict__ w3, long w_stride, T* __restrict__ out, long ldo,
                 int N, int K, const int* __restrict__ row_pair, int top, const int* __restrict__ tile_expert,
-                const int* __restrict__ tile_row0, const int* __restrict__ tile_n, const int* __restrict__ n_tiles) {
+                const int* __restrict__ tile_row0, const int* __restrict__ tile_n, const int* __restrict__ n_tiles,
+                const float* in_w) {
   if ((int)blockIdx.y >= *n_tiles) return;
   __shared__ float As[BK][BM + 4];
   __shared__ float W1s[BK][BN + 4];
@@ -563,12 +569,13 @@ moe_gemm_kernel(const T* x, long ldx, const T* __restrict__ w1, const T* __restr
   for (int i = 0; i < TM; ++i) {
     const int m = ty * TM + i;
     if (m >= rows) continue;
+    const float wgt = in_w != nullptr ? in_w[row_pair[row0 + m]] : 1.f;
 #pragma unroll
     for (int j = 0; j < TN; ++j) {
       const int n = n0 + tx * TN + j;
       if (n >= N) continue;
-      float v = acc[i][j];
-      if (GATED) v = v / (1.f + expf(-v)) * acc3[i][j];
+      float v = acc[i][j] * wgt;
+      if (GATED) v = v / (1.f + expf(-v)) * (acc3[i][j] * wgt);
       out[(size_t)(row0 + m) * ldo + n] = from_f32<T>(v);
     }
   }
@@ -578,13 +585,14 @@ extern "C" int fg_moe_gemm_tile_rows() { return BM; }
 
 extern "C" int fg_moe_gemm(const void* x, long ldx, const void* w1, const void* w3, long w_stride, void* out, long ldo, int dtype,
                            int N, int K, const int* row_pair, int top, const int* tile_expert, const int* tile_row0,
-                           const int* tile_n, const int* n_tiles, int max_tiles, cudaStream_t stream) {
+                           const int* tile_n, const int* n_tiles, int max_tiles, const float* in_w, cudaStream_t stream) {
   if (max_tiles == 0 || N == 0) return 0;
+  FG_CHECK_ARG(in_w == nullptr || row_pair != nullptr, "fg_moe_gemm: weights of the input need the rows' pairs");
   FG_CHECK_ARG(K > 0 && max_tiles <= 65535, "fg_moe_gemm: bad sizes K=%d tiles=%d", K, max_tiles);
   dim3 grid((N + BN - 1) / BN, max_tiles);
 #define LAUNCH(T, GATED)                                                                                         \
   moe_gemm_kernel<T, GATED><<<grid, 256, 0, stream>>>((const T*)x, ldx, (const T*)w1, (const T*)w3, w_stride, (T*)out, ldo, N, K, \
-                                                      row_pair, top, tile_expert, tile_row0, tile_n, n_tiles)
+                                                      row_pair, top, tile_expert, tile_row0, tile_n, n_tiles, in_w)
   if (dtype == FG_F32) {
     if (w3) LAUNCH(float, true); else LAUNCH(float, false);
   } else if (dtype == FG_BF16) {
@@ -635,7 +643,7 @@ moe_gemm_mma_kernel(const __nv_bfloat16* x, long ldx, const __nv_bfloat16* __res
                     const __nv_bfloat16* __restrict__ w3, long w_stride, __nv_bfloat16* __restrict__ out, long ldo, int N, int K,
                     const int* __restrict__ row_pair, int top, const int* __restrict__ tile_expert,
                     const int* __restrict__ tile_row0, const int* __restrict__ tile_n,
-                    const int* __restrict__ n_tiles) {
+                    const int* __restrict__ n_tiles, const float* in_w) {
   if ((int)blockIdx.y >= *n_tiles) return;
   extern __shared__ __align__(16) unsigned char moe_smem[];
   typedef __nv_bfloat16 (*Tile)[MM][MLD];  // MM == MN
@@ -711,6 +719,13 @@ moe_gemm_mma_kernel(const __nv_bfloat16* x, long ldx, const __nv_bfloat16* __res
     }
     __syncthreads();
   }
+  float row_w[2] = {1.f, 1.f};
+  if (in_w != nullptr)
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int m = warp * 16 + (lane >> 2) + half * 8;
+      if (m < rows) row_w[half] = in_w[row_pair[row0 + m]];
+    }
 #pragma unroll
   for (int nt = 0; nt < MN / 8; ++nt)
 #pragma unroll
@@ -718,10 +733,11 @@ moe_gemm_mma_kernel(const __nv_bfloat16* x, long ldx, const __nv_bfloat16* __res
       const int m = warp * 16 + (lane >> 2) + half * 8;
       const int n = n0 + nt * 8 + (lane & 3) * 2;
       if (m >= rows || n >= N) continue;
-      float v0 = acc[nt][half * 2], v1 = acc[nt][half * 2 + 1];
+      const float wgt = row_w[half];
+      float v0 = acc[nt][half * 2] * wgt, v1 = acc[nt][half * 2 + 1] * wgt;
       if (GATED) {
-        v0 = v0 / (1.f + expf(-v0)) * acc3[nt][half * 2];
-        v1 = v1 / (1.f + expf(-v1)) * acc3[nt][half * 2 + 1];
+        v0 = v0 / (1.f + expf(-v0)) * (acc3[nt][half * 2] * wgt);
+        v1 = v1 / (1.f + expf(-v1)) * (acc3[nt][half * 2 + 1] * wgt);
       }
       __nv_bfloat16* dst = out + (size_t)(row0 + m) * ldo + n;
       dst[0] = __float2bfloat16(v0);
@@ -733,8 +749,10 @@ extern "C" int fg_moe_mma_tile_rows() { return MM; }
 
 extern "C" int fg_moe_gemm_mma(const void* x, long ldx, const void* w1, const void* w3, long w_stride, void* out, long ldo, int N,
                                int K, const int* row_pair, int top, const int* tile_expert, const int* tile_row0,
-                               const int* tile_n, const int* n_tiles, int max_tiles, cudaStream_t stream) {
+                               const int* tile_n, const int* n_tiles, int max_tiles, const float* in_w,
+                               cudaStream_t stream) {
   if (max_tiles == 0 || N == 0) return 0;
+  FG_CHECK_ARG(in_w == nullptr || row_pair != nullptr, "fg_moe_gemm_mma: weights of the input need the rows' pairs");
   FG_CHECK_ARG(K > 0 && K % 8 == 0 && ldx % 8 == 0 && max_tiles <= 65535,
                "fg_moe_gemm_mma: bad sizes K=%d ldx=%ld tiles=%d", K, ldx, max_tiles);
   dim3 grid((N + MN - 1) / MN, max_tiles);
@@ -750,10 +768,10 @@ extern "C" int fg_moe_gemm_mma(const void* x, long ldx, const void* w1, const vo
   }
   if (w3)
     moe_gemm_mma_kernel<true><<<grid, 128, smem3, stream>>>((P)x, ldx, (P)w1, (P)w3, w_stride, (__nv_bfloat16*)out, ldo, N, K, row_pair,
-                                                        top, tile_expert, tile_row0, tile_n, n_tiles);
+                                                        top, tile_expert, tile_row0, tile_n, n_tiles, in_w);
   else
     moe_gemm_mma_kernel<false><<<grid, 128, smem2, stream>>>((P)x, ldx, (P)w1, nullptr, w_stride, (__nv_bfloat16*)out, ldo, N, K,
-                                                         row_pair, top, tile_expert, tile_row0, tile_n, n_tiles);
+                                                         row_pair, top, tile_expert, tile_row0, tile_n, n_tiles, in_w);
   FG_CHECK_LAUNCH("fg_moe_gemm_mma");
   return 0;
 }
@@ -771,7 +789,7 @@ __global__ void __launch_bounds__(fg_skinny::THREADS)
 moe_gemm_stream_kernel(const __nv_bfloat16* x, long ldx, const __nv_bfloat16* __restrict__ w1,
                        const __nv_bfloat16* __restrict__ w3, long w_stride, __nv_bfloat16* __restrict__ out, long ldo,
                        int N, int K, const int* row_pair, int top, const int* tile_expert, const int* tile_row0,
-                       const int* tile_n, const int* n_tiles, int act) {
+                       const int* tile_n, const int* n_tiles, int act, const float* in_w) {
   using namespace fg_skinny;
   extern __shared__ __align__(16) unsigned char ring_raw[];
   if ((int)blockIdx.y >= *n_tiles) return;
@@ -798,7 +816,8 @@ moe_gemm_stream_kernel(const __nv_bfloat16* x, long ldx, const __nv_bfloat16* __
     if (i >= 8 * 8) return;
     const int tok = i / 8, f = i - tok * 8;
     if (tok < rows && n0 + f < N) {
-      const float g = block_total<1>(red, f, tok), u = block_total<1>(red, f + 8, tok);
+      const float wgt = in_w != nullptr ? in_w[row_pair[row0 + tok]] : 1.f;
+      const float g = block_total<1>(red, f, tok) * wgt, u = block_total<1>(red, f + 8, tok) * wgt;
       out[(size_t)(row0 + tok) * ldo + n0 + f] = __float2bfloat16_rn(g / (1.f + expf(-g)) * u);
     }
   } else {
@@ -806,6 +825,7 @@ moe_gemm_stream_kernel(const __nv_bfloat16* x, long ldx, const __nv_bfloat16* __
       const int tok = i / ROWS, row = i - tok * ROWS;
       if (tok < rows && n0 + row < N) {
         float v = block_total<1>(red, row, tok);
+        if (in_w != nullptr) v *= in_w[row_pair[row0 + tok]];
         if (act != ACT_NONE) v = activate(__bfloat162float(__float2bfloat16_rn(v)), act);
         out[(size_t)(row0 + tok) * ldo + n0 + row] = __float2bfloat16_rn(v);
       }
@@ -818,9 +838,10 @@ extern "C" int fg_moe_stream_tile_rows() { return STREAM_ROWS; }
 extern "C" int fg_moe_gemm_stream(const void* x, long ldx, const void* w1, const void* w3, long w_stride, void* out,
                                   long ldo, int N, int K, const int* row_pair, int top, const int* tile_expert,
                                   const int* tile_row0, const int* tile_n, const int* n_tiles, int max_tiles, int act,
-                                  cudaStream_t stream) {
+                                  const float* in_w, cudaStream_t stream) {
   using namespace fg_skinny;
   if (max_tiles == 0 || N == 0) return 0;
+  FG_CHECK_ARG(in_w == nullptr || row_pair != nullptr, "fg_moe_gemm_stream: weights of the input need the rows' pairs");
   FG_CHECK_ARG(K > 0 && K % 8 == 0 && ldx % 8 == 0 && w_stride % 8 == 0 && max_tiles <= 65535,
                "fg_moe_gemm_stream: bad sizes K=%d ldx=%ld tiles=%d", K, ldx, max_tiles);
   FG_CHECK_ARG(((uintptr_t)x & 15) == 0 && ((uintptr_t)w1 & 15) == 0 && ((uintptr_t)w3 & 15) == 0,
@@ -841,11 +862,11 @@ extern "C" int fg_moe_gemm_stream(const void* x, long ldx, const void* w1, const
   if (w3)
     moe_gemm_stream_kernel<true, MODE><<<dim3((N + 7) / 8, max_tiles), THREADS, smem, stream>>>(
         (P)x, ldx, (P)w1, (P)w3, w_stride, (__nv_bfloat16*)out, ldo, N, K, row_pair, top, tile_expert, tile_row0, tile_n,
-        n_tiles, act);
+        n_tiles, act, in_w);
   else
     moe_gemm_stream_kernel<false, MODE><<<dim3((N + ROWS - 1) / ROWS, max_tiles), THREADS, smem, stream>>>(
         (P)x, ldx, (P)w1, nullptr, w_stride, (__nv_bfloat16*)out, ldo, N, K, row_pair, top, tile_expert, tile_row0, tile_n,
-        n_tiles, act);
+        n_tiles, act, in_w);
   FG_CHECK_LAUNCH("fg_moe_gemm_stream");
   return 0;
 }
@@ -861,7 +882,7 @@ moe_combine_kernel(const T* y, long ldy, const float* weights, const int* pair_r
     float acc = 0.f;
     for (int k = 0; k < top; ++k) {
       const int r = pair_row[(size_t)t * top + k];
-      if (r >= 0) acc = fmaf(weights[(size_t)t * top + k], to_f32<T>(y[(size_t)r * ldy + c]), acc);
+      if (r >= 0) acc = fmaf(weights ? weights[(size_t)t * top + k] : 1.f, to_f32<T>(y[(size_t)r * ldy + c]), acc);
     }
     if (shared != nullptr) acc = fmaf(g, to_f32<T>(shared[(size_t)t * lds + c]), acc);
     out[(size_t)t * ldo + c] = from_f32<T>(acc);
@@ -881,7 +902,7 @@ moe_combine_bf16x8_kernel(const __nv_bfloat16* y, long ldy, const float* weights
   const int t = blockIdx.x, piece = blockIdx.y * COMBINE_THREADS + threadIdx.x;
   for (int k = threadIdx.x; k < top; k += COMBINE_THREADS) {
     rows_s[k] = pair_row[(size_t)t * top + k];
-    w_s[k] = weights[(size_t)t * top + k];
+    w_s[k] = weights ? weights[(size_t)t * top + k] : 1.f;
   }
   const bool in = piece * 8 < dim;
   uint4 s4 = make_uint4(0u, 0u, 0u, 0u);

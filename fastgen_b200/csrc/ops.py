@@ -57,6 +57,8 @@ _CORE_SIGNATURES = {
     "fg_qk_head_factors": [_P, _L, _P, _L, _I, _I, _I, _I, _I, _I, _F, _F, _I, _P, _P, _P, _I, _P],
     "fg_mamba2_scan": [_P, _L, _P, _L, _L, _I, _P, _P, _P, _P, _L, _P, _L, _P, _P, _I, _I, _I, _I, _I, _P],
     "fg_gated_part_norm": [_P, _L, _P, _L, _I, _P, _P, _L, _P, _I, _I, _I, _F, _P],
+    "fg_selective_scan": [_P, _L, _P, _L, _P, _L, _P, _L, _L, _I, _P, _P, _P, _P, _L, _P, _L, _P, _P, _I, _I, _I, _P],
+    "fg_layer_norm_pair": [_P, _P, _P, _I, _I, _P, _P, _F, _P, _P, _F, _P, _I, _P, _I, _I, _P],
     "fg_rms_rows": [_P, _L, _I, _P, _F, _P, _L, _I, _I, _P],
     "fg_rotate_part": [_P, _L, _I, _P, _P, _P, _F, _I, _I, _I, _I, _I, _P],
     "fg_latent_prepare": [_P, _L, _I, _P, _F, _P, _F, _P, _P, _I, _I, _I, _P, _P, _I, _I, _I, _I, _P, _L, _P, _P, _L, _I, _I, _I,
@@ -65,20 +67,20 @@ _CORE_SIGNATURES = {
     "fg_latent_attention_simt": [_P, _I, _L, _L, _P, _L, _L, _P, _L, _L, _I, _P, _L, _P, _P, _I, _I, _I, _P, _P, _P,
                                  _P, _I, _I, _I, _I, _I, _F, _P, _P],
     "fg_rmsnorm": [_P, _I, _P, _I, _P, _I, _P, _I, _P, _I, _I, _F, _P],
-    "fg_silu_gate": [_P, _P, _I, _I, _I, _I, _P],
+    "fg_silu_gate": [_P, _P, _I, _I, _I, _I, _I, _P, _P, _P, _P],
     "fg_embedding_bigram": [_P, _P, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _P],
     "fg_dyt": [_P, _P, _I, _P, _P, _P, _P, _P, _P, _P, _I, _P, _I, _I, _P],
     "fg_bias_act": [_P, _P, _I, _I, _I, _I, _P],
     "fg_scale_softcap": [_P, _I, _I, _F, _F, _P],
     "fg_rope_kv_write": [_P, _I, _P, _I, _P, _I, _I, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P, _P,
-                         _P, _I, _P],
+                         _P, _I, _F, _I, _P],
     "fg_qk_rstd": [_P, _L, _I, _I, _P, _L, _I, _I, _I, _P, _F, _P, _I, _P],
     "fg_rmsnorm_sum": [_P, _P, _P, _I, _I, _P, _P, _I, _I, _P, _I, _P, _I, _I, _F, _P],
     "fg_part_norm": [_P, _I, _P, _I, _P, _P, _P, _I, _P, _I, _I, _I, _F, _P],
     "fg_gemm_f32_nt_from": [_P, _I, _I, _P, _I, _P, _I, _I, _I, _I, _P],
     "fg_gemm_f32_nt": [_P, _I, _P, _I, _P, _I, _I, _I, _I, _P, _P],
     "fg_gemm_skinny_bf16": [_P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _P, _I, _P],
-    "fg_gemm_skinny_swiglu_bf16": [_P, _I, _P, _I, _P, _I, _I, _I, _I, _P],
+    "fg_gemm_skinny_swiglu_bf16": [_P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _P],
     "fg_gemm_skinny_qkv_bf16": [_P, _I, _P, _I, _P, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I,
                                 _I, _I, _P, _P],
     "fg_sample": [_P, _I, _I, _I, _P, _F, c_ulonglong, _P, _P, _P, _P, _P, _P, _P],
@@ -122,6 +124,9 @@ SIGMOID_DECODE_KEYS = 256  # key positions per stretch of the sigmoid attention'
 
 #: activations the products' epilogues and ``bias_act`` know
 ACTIVATIONS = {None: 0, "none": 0, "gelu_erf": 1, "gelu_tanh": 2, "relu2": 3}
+
+#: activations of a gated feed-forward's gate
+GATES = {"silu": 0, "relu": 1}
 
 
 def _declare(lib: ctypes.CDLL, signatures) -> None:
@@ -195,9 +200,9 @@ def latent(rank: int, rot_dim: int):
 
 
 _DELTA_SIGNATURES = {
-    "fg_delta_scan": [_P, _L, _P, _L, _P, _L, _I, _P, _P, _P, _L, _P, _L, _P, _P, _I, _P, _I, _P, _I, _I, _I, _I, _P],
+    "fg_delta_scan": [_P, _L, _P, _L, _P, _L, _I, _P, _P, _P, _L, _P, _L, _P, _P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _P],
     "fg_delta_scan_scratch_floats": [_I, _I, _I, _I, _I],
-    "fg_head_norm_gate": [_P, _L, _P, _L, _I, _P, _P, _L, _P, _I, _I, _I, _F, _P],
+    "fg_head_norm_gate": [_P, _L, _P, _L, _I, _P, _P, _L, _P, _I, _I, _I, _F, _I, _P],
 }
 _MOE_SIGNATURES = {
     "fg_moe_logits": [_P, _I, _L, _P, _L, _P, _P, _P, _I, _I, _I, _P],
@@ -205,9 +210,9 @@ _MOE_SIGNATURES = {
     "fg_moe_route_groups": [_P, _L, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _P],
     "fg_moe_plan": [_P, _I, _I, _I, _P, _P, _P, _P, _P, _P, _I, _P, _P],
     "fg_moe_gather": [_P, _L, _P, _L, _I, _P, _P, _I, _I, _I, _I, _P],
-    "fg_moe_gemm": [_P, _L, _P, _P, _L, _P, _L, _I, _I, _I, _P, _I, _P, _P, _P, _P, _I, _P],
-    "fg_moe_gemm_mma": [_P, _L, _P, _P, _L, _P, _L, _I, _I, _P, _I, _P, _P, _P, _P, _I, _P],
-    "fg_moe_gemm_stream": [_P, _L, _P, _P, _L, _P, _L, _I, _I, _P, _I, _P, _P, _P, _P, _I, _I, _P],
+    "fg_moe_gemm": [_P, _L, _P, _P, _L, _P, _L, _I, _I, _I, _P, _I, _P, _P, _P, _P, _I, _P, _P],
+    "fg_moe_gemm_mma": [_P, _L, _P, _P, _L, _P, _L, _I, _I, _P, _I, _P, _P, _P, _P, _I, _P, _P],
+    "fg_moe_gemm_stream": [_P, _L, _P, _P, _L, _P, _L, _I, _I, _P, _I, _P, _P, _P, _P, _I, _I, _P, _P],
     "fg_moe_combine": [_P, _L, _P, _P, _P, _L, _P, _L, _P, _L, _I, _I, _I, _I, _P],
 }
 _RECUR_SIGNATURES = {
@@ -450,6 +455,50 @@ class Ops:
         _check(self.lib, self.lib.fg_gated_part_norm(
             _ptr(y), y.stride(0), _ptr(z), z.stride(0), _code(z.dtype), _ptr(weight), _ptr(out), out.stride(0),
             _ptr(ctx.req), t, width, parts, float(eps), _stream()))
+        return out
+
+    # -- the selective state-space mixer ------------------------------------------------------------
+    def selective_scan(self, x, dt, low, b_offset: int, z, dt_bias, a_log2, d_skip, state, ctx,
+                       n_state: int) -> torch.Tensor:
+        """``S[c, n] <- exp2(d_c a_log2[c, n]) S[c, n] + d_c x_c B_n``, ``y_c = sum_n S[c, n] C_n + D_c x_c`` with
+        ``d = softplus(dt + dt_bias)``, token by token in float32 per (sequence, channel), from and into ``state``
+        [slots, .] (its first ``inner * n_state`` numbers); returns ``y * silu(z)`` [T, inner].  ``x``, ``dt``,
+        ``z`` [T, inner] and ``low`` (B in the ``n_state`` columns from ``b_offset``, C behind it) are row-strided
+        views of the compute dtype, which the result has; ``a_log2`` [inner, n_state] is ``A`` times ``log2 e``."""
+        t, inner = x.shape
+        for v in (x, dt, z, low):
+            assert v.dtype == x.dtype and v.stride(1) == 1 and v.shape[0] == t
+        assert dt.shape == z.shape == x.shape and low.shape[1] >= b_offset + 2 * n_state
+        for v, size in ((dt_bias, inner), (d_skip, inner), (a_log2, inner * n_state)):
+            assert v.dtype == torch.float32 and v.numel() == size and v.is_contiguous()
+        assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1] >= inner * n_state
+        out = torch.empty((t, inner), dtype=x.dtype, device=x.device)
+        _check(self.lib, self.lib.fg_selective_scan(
+            _ptr(x), x.stride(0), _ptr(dt), dt.stride(0), _ptr(z), z.stride(0), _ptr(low), low.stride(0), int(b_offset),
+            _code(x.dtype), _ptr(dt_bias), _ptr(a_log2), _ptr(d_skip), _ptr(out), out.stride(0), _ptr(state),
+            state.stride(0), _ptr(ctx.seq_slot), _ptr(ctx.seq_start), ctx.n_seqs, inner, n_state, _stream()))
+        return out
+
+    def layer_norm_pair(self, h, terms, close_w, close_b, close_eps: float, w, b, eps: float, out, rows=None):
+        """``h += norm(sum_i coef_i * delta_i) * close_w + close_b`` (float32), then ``out = norm(h) * w + b``, both
+        norms with mean and variance: the norm that closes a sub-layer, the residual sum and the norm that
+        opens the next one.  ``terms`` is a sequence of one to four ``(delta [T, dim], coef)`` of one dtype; the
+        biases may be ``None``.  With ``rows`` only those rows are computed and ``h`` stays as it was."""
+        assert h.is_contiguous() and h.dtype == torch.float32 and h.dim() == 2
+        dim = h.shape[1]
+        n = h.shape[0] if rows is None else rows.numel()
+        terms = list(terms)
+        assert 1 <= len(terms) <= 4 and len({d.dtype for d, _ in terms}) == 1
+        for d, _ in terms:
+            assert d.is_contiguous() and d.shape == h.shape
+        for v in (close_w, close_b, w, b):
+            assert v is None or (v.dtype == torch.float32 and v.is_contiguous() and v.numel() == dim)
+        assert out.is_contiguous() and out.shape == (n, dim) and (rows is None or rows.dtype == torch.int32)
+        ptrs = (c_void_p * len(terms))(*[d.data_ptr() for d, _ in terms])
+        coefs = (c_float * len(terms))(*[float(c) for _, c in terms])
+        _check(self.lib, self.lib.fg_layer_norm_pair(
+            _ptr(h), ptrs, coefs, len(terms), _code(terms[0][0].dtype), _ptr(close_w), _ptr(close_b), float(close_eps),
+            _ptr(w), _ptr(b), float(eps), _ptr(out), _code(out.dtype), _ptr(rows), n, dim, _stream()))
         return out
 
     # -- latent attention ---------------------------------------------------------------------------
@@ -754,20 +803,23 @@ class Ops:
         ``offset .. + channels`` of ``proj`` (see ``mamba2_conv``): float32 [T, channels]."""
         return self.mamba2_conv(proj, offset, channels, weight, None, state, conv_offset, taps, ctx)
 
-    def delta_scan(self, qkv, a, b, dt_bias, a_log, state, ctx, heads: int, kv_heads: int, d: int, dv: int):
+    def delta_scan(self, qkv, a, b, dt_bias, a_log, state, ctx, heads: int, kv_heads: int, d: int, dv: int,
+                   head_decay: bool = False):
         """The gated delta rule per (sequence, head), token by token in float32, from and into ``state``
         [slots, .] (a slot's first ``heads * dv * d`` numbers, laid out [heads][dv][d]):
         ``S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q`` with q, k made unit vectors
         (q also times ``d ** -0.5``), ``g = exp(-exp(a_log) softplus(a + dt_bias))``, ``beta =
-        sigmoid(b)``.  ``qkv`` float32 [T, q | k | v] (``kv_heads * d`` twice, ``heads * dv``); ``a``
+        sigmoid(b)``.  With ``head_decay`` there is one decay per head: ``a`` [T, heads], ``dt_bias`` [heads].
+        ``qkv`` float32 [T, q | k | v] (``kv_heads * d`` twice, ``heads * dv``); ``a``
         [T, heads * d] and ``b`` [T, heads] strided views of the compute dtype.  Returns o float32
         [T, heads * dv]."""
         lib = delta_rule()
         t = qkv.shape[0]
+        decays = heads if head_decay else heads * d
         assert qkv.dtype == torch.float32 and qkv.stride(1) == 1 and qkv.shape[1] == 2 * kv_heads * d + heads * dv
-        assert a.stride(1) == 1 and b.stride(1) == 1 and a.dtype == b.dtype and a.shape == (t, heads * d)
+        assert a.stride(1) == 1 and b.stride(1) == 1 and a.dtype == b.dtype and a.shape == (t, decays)
         assert b.shape == (t, heads) and state.dtype == torch.float32 and state.is_contiguous()
-        assert dt_bias.dtype == torch.float32 and dt_bias.numel() == heads * d and dt_bias.is_contiguous()
+        assert dt_bias.dtype == torch.float32 and dt_bias.numel() == decays and dt_bias.is_contiguous()
         assert a_log.dtype == torch.float32 and a_log.numel() == heads and a_log.is_contiguous()
         out = torch.empty((t, heads * dv), dtype=torch.float32, device=qkv.device)
         # the tokens as the recurrence reads them (unit vectors, decays, step sizes; padded rows)
@@ -776,12 +828,13 @@ class Ops:
         _check(lib, lib.fg_delta_scan(
             _ptr(qkv), qkv.stride(0), _ptr(a), a.stride(0), _ptr(b), b.stride(0), _code(a.dtype), _ptr(dt_bias),
             _ptr(a_log), _ptr(out), out.stride(0), _ptr(state), state.stride(0), _ptr(ctx.seq_slot),
-            _ptr(ctx.seq_start), ctx.n_seqs, _ptr(ctx.req), t, _ptr(scratch), heads, kv_heads, d, dv, _stream()))
+            _ptr(ctx.seq_start), ctx.n_seqs, _ptr(ctx.req), t, _ptr(scratch), heads, kv_heads, d, dv,
+            int(head_decay), _stream()))
         Ops.launches += 1  # the kernel that prepares the tokens
         return out
 
-    def head_norm_gate(self, o, z, weight, heads: int, dv: int, eps: float, ctx) -> torch.Tensor:
-        """Per head ``o * rsqrt(mean(o^2) + eps) * weight * sigmoid(z)``: ``o`` float32 [T, heads * dv],
+    def head_norm_gate(self, o, z, weight, heads: int, dv: int, eps: float, ctx, act: str = "sigmoid") -> torch.Tensor:
+        """Per head ``o * rsqrt(mean(o^2) + eps) * weight * act(z)`` (``act``: ``"sigmoid"`` or ``"silu"``): ``o`` float32 [T, heads * dv],
         ``z`` of the compute dtype (which the result has), ``weight`` float32 [dv] shared by the heads."""
         lib = delta_rule()
         t = o.shape[0]
@@ -790,7 +843,7 @@ class Ops:
         out = torch.empty((t, heads * dv), dtype=z.dtype, device=o.device)
         _check(lib, lib.fg_head_norm_gate(
             _ptr(o), o.stride(0), _ptr(z), z.stride(0), _code(z.dtype), _ptr(weight), _ptr(out), out.stride(0),
-            _ptr(ctx.req), t, heads, dv, float(eps), _stream()))
+            _ptr(ctx.req), t, heads, dv, float(eps), {"sigmoid": 0, "silu": 1}[act], _stream()))
         return out
 
     # -- routed experts -----------------------------------------------------------------------------
@@ -836,7 +889,7 @@ class Ops:
         return ids, weights
 
     def moe_experts(self, x, ids, weights, w1, w3, w2, w13=None, act: Optional[str] = None, shared=None,
-                    shared_gate=None) -> torch.Tensor:
+                    shared_gate=None, weigh_input: bool = False) -> torch.Tensor:
         """``sum_k weights[t, k] * expert_{ids[t, k]}(x[t])`` with expert ``e`` the gated feed-forward
         ``w2[e] (silu(w1[e] x) * (w3[e] x))``; ``w1``, ``w3`` [E, F, K] (each expert's matrix contiguous,
         the experts a fixed stride apart: they may be the halves of ``w13`` [E, 2F, K]) and ``w2``
@@ -852,7 +905,10 @@ class Ops:
         ``ACTIVATIONS`` (``w13`` is then ``w1`` itself, for the grouped product).
 
         ``shared`` [T, K]: a further summand of every token; with ``shared_gate`` (float32 [T], strided) it
-        is multiplied by ``sigmoid(shared_gate[t])``.  Both join in the kernel that sums the experts."""
+        is multiplied by ``sigmoid(shared_gate[t])``.  Both join in the kernel that sums the experts.
+
+        ``weigh_input``: a weight multiplies the expert's input instead, ``sum_k expert(weights[t, k] * x[t])``:
+        the first products' sums are multiplied by it before the gate (or the activation)."""
         lib = moe()
         t, k = x.shape
         n_experts, f, _ = w1.shape
@@ -865,7 +921,8 @@ class Ops:
         assert gated or ACTIVATIONS[act] >= 0
         w_stride = w1.stride(0)
         grouped = (w13 is not None and x.dtype == torch.bfloat16 and pairs >= MOE_GROUPED_PAIRS and k % 8 == 0
-                   and f % 8 == 0 and hasattr(torch, "_grouped_mm") and not os.environ.get("FG_NO_GROUPED_MM"))
+                   and f % 8 == 0 and hasattr(torch, "_grouped_mm") and not os.environ.get("FG_NO_GROUPED_MM")
+                   and (gated or not weigh_input))
         mma = (not grouped and x.dtype == torch.bfloat16 and k % 8 == 0 and f % 8 == 0 and x.stride(0) % 8 == 0
                and w_stride % 8 == 0 and x.data_ptr() % 16 == 0 and w1.data_ptr() % 16 == 0
                and (not gated or w3.data_ptr() % 16 == 0) and hasattr(lib, "fg_moe_gemm_mma") and not os.environ.get("FG_NO_MOE_MMA"))
@@ -891,7 +948,10 @@ class Ops:
             h = torch._grouped_mm(xs, w13.transpose(1, 2), offs=expert_end)
             if gated:
                 mid = torch.empty((pairs, f), dtype=x.dtype, device=x.device)
-                self.silu_gate(h, mid, 0)
+                if weigh_input:
+                    self.silu_gate(h, mid, 0, row_scale=weights, row_index=row_pair, n_rows=expert_end[-1:])
+                else:
+                    self.silu_gate(h, mid, 0)
             else:
                 mid = self.bias_act(h, act)
             y = torch._grouped_mm(mid, w2.transpose(1, 2), offs=expert_end)
@@ -899,34 +959,35 @@ class Ops:
             # (rows beyond the plan's last tile are never written; zeroed where a kernel reads them all)
             mid = (torch.empty if gated else torch.zeros)((pairs, f), dtype=x.dtype, device=x.device)
             y = torch.empty((pairs, k), dtype=x.dtype, device=x.device)
-            tiles = (_ptr(tile_expert), _ptr(tile_row0), _ptr(tile_n), _ptr(n_tiles), max_tiles, _stream())
+            tiles = (_ptr(tile_expert), _ptr(tile_row0), _ptr(tile_n), _ptr(n_tiles), max_tiles)
+            in_w = _ptr(weights) if weigh_input else None
             if stream:
                 # a few rows an expert: the matrices are streamed once, the activation is an epilogue
                 _check(lib, lib.fg_moe_gemm_stream(_ptr(x), x.stride(0), _ptr(w1), _ptr(w3), w_stride, _ptr(mid),
-                                                   mid.stride(0), f, k, _ptr(row_pair), top, *tiles[:-1],
-                                                   0 if gated else ACTIVATIONS[act], tiles[-1]))
+                                                   mid.stride(0), f, k, _ptr(row_pair), top, *tiles,
+                                                   0 if gated else ACTIVATIONS[act], in_w, _stream()))
                 _check(lib, lib.fg_moe_gemm_stream(_ptr(mid), mid.stride(0), _ptr(w2), None, w2.stride(0), _ptr(y),
-                                                   y.stride(0), k, f, None, top, *tiles[:-1], 0, tiles[-1]))
+                                                   y.stride(0), k, f, None, top, *tiles, 0, None, _stream()))
             elif mma:
                 _check(lib, lib.fg_moe_gemm_mma(_ptr(x), x.stride(0), _ptr(w1), _ptr(w3), w_stride, _ptr(mid),
-                                                mid.stride(0), f, k, _ptr(row_pair), top, *tiles))
+                                                mid.stride(0), f, k, _ptr(row_pair), top, *tiles, in_w, _stream()))
                 if not gated:
                     self.bias_act(mid, act)
                 _check(lib, lib.fg_moe_gemm_mma(_ptr(mid), mid.stride(0), _ptr(w2), None, w2.stride(0), _ptr(y),
-                                                y.stride(0), k, f, None, top, *tiles))
+                                                y.stride(0), k, f, None, top, *tiles, None, _stream()))
             else:
                 code = _code(x.dtype)
                 _check(lib, lib.fg_moe_gemm(_ptr(x), x.stride(0), _ptr(w1), _ptr(w3), w_stride, _ptr(mid), mid.stride(0),
-                                            code, f, k, _ptr(row_pair), top, *tiles))
+                                            code, f, k, _ptr(row_pair), top, *tiles, in_w, _stream()))
                 if not gated:
                     self.bias_act(mid, act)
                 _check(lib, lib.fg_moe_gemm(_ptr(mid), mid.stride(0), _ptr(w2), None, w2.stride(0), _ptr(y), y.stride(0),
-                                            code, k, f, None, top, *tiles))
+                                            code, k, f, None, top, *tiles, None, _stream()))
         out = torch.empty((t, k), dtype=x.dtype, device=x.device)
         assert shared is None or (shared.shape == (t, k) and shared.dtype == x.dtype and shared.stride(1) == 1)
         assert shared_gate is None or (shared is not None and shared_gate.dtype == torch.float32 and shared_gate.shape == (t,))
         _check(lib, lib.fg_moe_combine(
-            _ptr(y), y.stride(0), _ptr(weights), _ptr(pair_row), _ptr(shared), shared.stride(0) if shared is not None else 0,
+            _ptr(y), y.stride(0), None if weigh_input else _ptr(weights), _ptr(pair_row), _ptr(shared), shared.stride(0) if shared is not None else 0,
             _ptr(shared_gate), shared_gate.stride(0) if shared_gate is not None else 0, _ptr(out), out.stride(0),
             _code(x.dtype), t, k, top, _stream()))
         return out
@@ -988,8 +1049,8 @@ class Ops:
                 and x.stride(0) % 8 == 0 and w.stride(0) % 8 == 0 and x.stride(1) == 1 and w.stride(1) == 1
                 and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
 
-    def linear_swiglu(self, x: torch.Tensor, w13: torch.Tensor) -> Optional[torch.Tensor]:
-        """``silu(x @ w1.T) * (x @ w3.T)`` in one kernel for a few tokens, for
+    def linear_swiglu(self, x: torch.Tensor, w13: torch.Tensor, act: str = "silu") -> Optional[torch.Tensor]:
+        """``act(x @ w1.T) * (x @ w3.T)`` (``act`` a key of ``GATES``) in one kernel for a few tokens, for
         ``w13`` that holds w1 and w3 interleaved in blocks of 8 rows; ``None``
         when the shapes do not allow it (the caller then runs the product and
         the gate separately)."""
@@ -999,7 +1060,7 @@ class Ops:
             return None
         out = torch.empty((m, f), dtype=torch.bfloat16, device=x.device)
         _check(self.lib, self.lib.fg_gemm_skinny_swiglu_bf16(
-            _ptr(x), x.stride(0), _ptr(w13), w13.stride(0), _ptr(out), out.stride(0), m, f, k, _stream()))
+            _ptr(x), x.stride(0), _ptr(w13), w13.stride(0), _ptr(out), out.stride(0), m, f, k, GATES[act], _stream()))
         return out
 
     def qkv_rope_write(self, x, wqkv, pos, req, freqs, memory, n_heads: int, n_kv_heads: int,
@@ -1020,24 +1081,30 @@ class Ops:
             memory.k_pages.shape[0], n_heads, n_kv_heads, head_dim, _ptr(self.status), _stream()))
         return q
 
-    def silu_gate(self, x13: torch.Tensor, out: torch.Tensor, interleave: int = 0) -> torch.Tensor:
-        """``silu(gate) * up`` for ``x13`` holding gate and up as halves
-        (``interleave=0``) or interleaved in blocks of 8 columns (``8``)."""
+    def silu_gate(self, x13: torch.Tensor, out: torch.Tensor, interleave: int = 0, act: str = "silu", row_scale=None,
+                  row_index=None, n_rows=None) -> torch.Tensor:
+        """``act(gate) * up`` (``act`` a key of ``GATES``) for ``x13`` holding gate and up as halves
+        (``interleave=0``) or interleaved in blocks of 8 columns (``8``).  With ``row_scale`` (float32) row
+        ``t``'s gate and up are first multiplied by ``row_scale[row_index[t]]``, and only the first
+        ``n_rows[0]`` rows (a device int) are computed."""
         n, two_f = x13.shape
         assert x13.is_contiguous() and out.is_contiguous() and out.shape == (n, two_f // 2)
         _check(self.lib, self.lib.fg_silu_gate(_ptr(x13), _ptr(out), _code(x13.dtype), n, two_f // 2,
-                                               interleave, _stream()))
+                                               interleave, GATES[act], _ptr(row_scale), _ptr(row_index), _ptr(n_rows),
+                                               _stream()))
         return out
 
     def rope_kv_write(self, q, k, v, pos, req, freqs, k_pages, v_pages, block_table,
-                      page_size: int, n_heads: int, n_kv_heads: int, head_dim: int, v_freqs=None, qk_norm=None) -> None:
+                      page_size: int, n_heads: int, n_kv_heads: int, head_dim: int, v_freqs=None, qk_norm=None,
+                      magnitude: float = 1.0, rot_pairs: int = 0) -> None:
         """Rotate ``q`` in place; rotate ``k`` and copy ``v`` into their pages (``v`` is
         rotated too, by the table ``v_freqs``, when that is given).
         ``q``/``k``/``v`` are row-strided views [T, heads*head_dim]; ``k``/``v``
         may both be ``None`` (queries only).  ``qk_norm`` = (rstd [T, 2], query weights, key
         weights), all float32: queries and keys are multiplied by their token's factor (see
         ``qk_rstd``) and their weights before they turn.  An ``rstd`` of [T, heads + kv heads] holds a
-        factor per head instead (see ``qk_head_factors``); the weights may then be ``None`` (ones)."""
+        factor per head instead (see ``qk_head_factors``); the weights may then be ``None`` (ones).
+        ``magnitude`` multiplies cosine and sine of a head's first ``rot_pairs`` pairs of queries and keys."""
         rstd, qn_w, kn_w = qk_norm if qk_norm is not None else (None, None, None)
         rstd_heads = 0
         if rstd is not None:
@@ -1064,7 +1131,7 @@ class Ops:
             _ptr(v_pages) if k is not None else None,
             _ptr(block_table) if k is not None else None, width, page_size, n_pages,
             t, n_heads, n_kv_heads, head_dim, _ptr(self.status), _ptr(rstd), _ptr(qn_w), _ptr(kn_w), rstd_heads,
-            _stream()))
+            float(magnitude), int(rot_pairs), _stream()))
 
     def qk_head_factors(self, q, k, pos, req, n_heads: int, n_kv_heads: int, head_dim: int, real_dim: int,
                         norm_eps: Optional[float] = None, temp=None) -> torch.Tensor:
@@ -1255,7 +1322,7 @@ class Ops:
     def attention(self, q, out, memory, ctx, n_heads: int, n_kv_heads: int, head_dim: int,
                   window: Optional[int], scale: float, out_freqs: Optional[torch.Tensor] = None,
                   keep_first: int = 0, softcap: Optional[float] = None,
-                  sinks: Optional[torch.Tensor] = None) -> bool:
+                  sinks: Optional[torch.Tensor] = None, chunk: Optional[int] = None) -> bool:
         """Paged causal attention of the step's query tokens; ``memory`` is the
         run's :class:`~fastgen_b200.cache.LayerMemory`, ``ctx`` the step's
         context.  bfloat16 runs on the tensor cores: prompt portions in one
@@ -1270,21 +1337,25 @@ class Ops:
         ``softcap``: a scaled score ``s`` enters the softmax as ``softcap * tanh(s / softcap)``.
 
         ``sinks`` (float32 [heads] or ``None``): ``exp(sinks[h])`` joins the softmax's denominator of head
-        ``h`` once; it has no key and no value and is not scaled."""
+        ``h`` once; it has no key and no value and is not scaled.
+
+        ``chunk`` (excludes a window): a query sees only the keys of its own chunk of that many positions."""
         lib = attn(head_dim)
+        assert not (window and chunk)
+        window = -int(chunk) if chunk else int(window or 0)  # (see first_visible in common.cuh)
         assert sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == n_heads and sinks.is_contiguous())
         k_pages, v_pages, block_table, page_size = (
             memory.k_pages, memory.v_pages, memory.block_table, memory.page_size)
         assert q.stride(1) == 1 and out.stride(1) == 1
         common = (_ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.shape[1], page_size,
                   k_pages.shape[0], _ptr(ctx.pos))
-        keep_first = int(keep_first) if window else 0
+        keep_first = int(keep_first) if window > 0 else 0
         if q.dtype == torch.float32:
             tiles = ctx.attention_tiles(attention_tiling(n_heads, n_kv_heads, SIMT_ROWS), 1)
             _check(lib, lib.fg_attention_simt(
                 _ptr(q), q.stride(0), _ptr(out), out.stride(0), _code(q.dtype), *common,
                 _ptr(tiles.req), _ptr(tiles.tok0), _ptr(tiles.ntok), tiles.n,
-                n_heads, n_kv_heads, head_dim, int(window or 0), keep_first, float(scale), float(softcap or 0.0),
+                n_heads, n_kv_heads, head_dim, window, keep_first, float(scale), float(softcap or 0.0),
                 _ptr(sinks), _ptr(self.status), _stream()))
             return False
         # windows that keep a sequence's first positions visible run on the mma.sync kernels (on TMA
@@ -1307,7 +1378,7 @@ class Ops:
             args = (_ptr(q), q.stride(0), _ptr(out), out.stride(0), memory.tensor_maps[2].ptr,
                     memory.tensor_maps[3].ptr, memory.layer_index, _ptr(block_table), block_table.shape[1],
                     page_size, k_pages.shape[0], _ptr(ctx.pos), _ptr(tiles.req), _ptr(tiles.tok0),
-                    _ptr(tiles.ntok), tiles.n, n_heads, n_kv_heads, head_dim, int(window or 0), float(scale))
+                    _ptr(tiles.ntok), tiles.n, n_heads, n_kv_heads, head_dim, window, float(scale))
             if tc5:
                 max_keys = -1 if tiles.max_keys is None else tiles.max_keys
                 # a captured list has padding: what a step of prompt tokens only would hold
@@ -1323,7 +1394,7 @@ class Ops:
             _check(lib, lib.fg_attention_prefill_bf16(
                 _ptr(q), q.stride(0), _ptr(out), out.stride(0), *common,
                 _ptr(tiles.req), _ptr(tiles.tok0), _ptr(tiles.ntok), tiles.n,
-                n_heads, n_kv_heads, head_dim, int(window or 0), keep_first, float(scale), float(softcap or 0.0),
+                n_heads, n_kv_heads, head_dim, window, keep_first, float(scale), float(softcap or 0.0),
                 _ptr(sinks), _ptr(self.status), _stream()))
         singles = ctx.single_tokens()
         fused = out_freqs is not None and tiles.n == 0 and singles.n > 0
@@ -1340,7 +1411,7 @@ class Ops:
             floats = lib.fg_attention_decode_scratch_floats(singles.n, max_splits, n_heads, pairs)
             scratch = self._decode_scratch(floats)
             head = (_ptr(singles.req), _ptr(singles.tok), singles.n, n_heads, n_kv_heads, head_dim,
-                    int(window or 0), float(scale), _ptr(scratch), scratch.numel(), max_splits)
+                    window, float(scale), _ptr(scratch), scratch.numel(), max_splits)
             if not tma:
                 head = head[:7] + (keep_first,) + head[7:]
             if tma:

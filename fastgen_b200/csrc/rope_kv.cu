@@ -11,6 +11,8 @@
 // of a pool laid out [n_pages, n_kv_heads, page, head_dim], so that the
 // [page, head_dim] tile of one head is contiguous.
 // Tokens whose request index is negative are padding: nothing is written.
+// A magnitude other than 1 multiplies cosine and sine of the first `rot_pairs` pairs of queries and keys (the
+// pairs that turn: dimensions that pass unchanged keep their size).
 #include "common.cuh"
 
 constexpr int ROPE_THREADS = 128;
@@ -54,7 +56,7 @@ rope_kv_kernel(T* __restrict__ q, int q_stride, const T* __restrict__ k, int k_s
                const float* __restrict__ v_freqs, T* __restrict__ k_pages, T* __restrict__ v_pages, const int* __restrict__ block_table, int table_width,
                int page_size, int n_pages, int n_heads, int n_kv_heads, int head_dim, int* status,
                bool vec, int heads_per_block, const float* rstd, const float* __restrict__ qn_w,
-               const float* __restrict__ kn_w, int rstd_heads) {
+               const float* __restrict__ kn_w, int rstd_heads, float magnitude, int rot_pairs) {
   const int t = blockIdx.x;
   const int r = req[t];
   if (r < 0) return;
@@ -70,7 +72,13 @@ rope_kv_kernel(T* __restrict__ q, int q_stride, const T* __restrict__ k, int k_s
   // queries and keys normed over their whole projection: the token's two factors; with rstd_heads
   // (= query heads + key heads) every head of the token has a factor of its own
   const float rq = rstd && !rstd_heads ? rstd[2 * t] : 1.f, rk = rstd && !rstd_heads ? rstd[2 * t + 1] : 1.f;
-  if (freqs != nullptr) sincosf((float)p * freqs[j], &s, &c);
+  if (freqs != nullptr) {
+    sincosf((float)p * freqs[j], &s, &c);
+    if (j < rot_pairs) {
+      s *= magnitude;
+      c *= magnitude;
+    }
+  }
   if (v_freqs != nullptr) sincosf((float)p * v_freqs[j], &sv, &cv);
   size_t slot = 0;
   bool have_slot = false;
@@ -130,7 +138,7 @@ rope_kv_bf16x8_kernel(__nv_bfloat16* __restrict__ q, int q_stride, const __nv_bf
                       const int* __restrict__ block_table, int table_width, int page_size, int n_pages,
                       int n_heads, int n_kv_heads, int head_dim, int* status, int heads_per_block,
                       const float* rstd, const float* __restrict__ qn_w, const float* __restrict__ kn_w,
-                      int rstd_heads) {
+                      int rstd_heads, float magnitude, int rot_pairs) {
   const int t = blockIdx.x;
   const int r = req[t];
   if (r < 0) return;
@@ -147,7 +155,13 @@ rope_kv_bf16x8_kernel(__nv_bfloat16* __restrict__ q, int q_stride, const __nv_bf
   for (int i = 0; i < 4; ++i) {
     sn[i] = snv[i] = 0.f;
     cs[i] = csv[i] = 1.f;
-    if (freqs != nullptr) sincosf((float)p * freqs[piece * 4 + i], &sn[i], &cs[i]);
+    if (freqs != nullptr) {
+      sincosf((float)p * freqs[piece * 4 + i], &sn[i], &cs[i]);
+      if (piece * 4 + i < rot_pairs) {
+        sn[i] *= magnitude;
+        cs[i] *= magnitude;
+      }
+    }
     if (v_freqs != nullptr) sincosf((float)p * v_freqs[piece * 4 + i], &snv[i], &csv[i]);
   }
   size_t slot = 0;
@@ -373,7 +387,7 @@ extern "C" int fg_rope_kv_write(void* q, int q_stride, const void* k, int k_stri
                                 const int* block_table, int table_width, int page_size, int n_pages,
                                 int n_tokens, int n_heads, int n_kv_heads, int head_dim, int* status,
                                 const float* rstd, const float* qn_w, const float* kn_w, int rstd_heads,
-                                cudaStream_t stream) {
+                                float magnitude, int rot_pairs, cudaStream_t stream) {
   // rstd: null, or float32 factors by which queries and keys are multiplied before they turn: [T, 2]
   // (a token's queries, its keys) when rstd_heads is 0, else [T, rstd_heads] with rstd_heads = n_heads +
   // n_kv_heads (every query head, then every key head).  qn_w / kn_w: per-column weights that join the
@@ -403,7 +417,7 @@ extern "C" int fg_rope_kv_write(void* q, int q_stride, const void* k, int k_stri
     rope_kv_bf16x8_kernel<<<grid, threads, 0, stream>>>(
         (__nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)k, k_stride, (const __nv_bfloat16*)v, v_stride, pos, req,
         freqs, v_freqs, (__nv_bfloat16*)k_pages, (__nv_bfloat16*)v_pages, block_table, table_width, page_size,
-        n_pages, n_heads, n_kv_heads, head_dim, status, ipt, rstd, qn_w, kn_w, rstd_heads);
+        n_pages, n_heads, n_kv_heads, head_dim, status, ipt, rstd, qn_w, kn_w, rstd_heads, magnitude, rot_pairs);
     FG_CHECK_LAUNCH("fg_rope_kv_write");
     return 0;
   }
@@ -411,12 +425,12 @@ extern "C" int fg_rope_kv_write(void* q, int q_stride, const void* k, int k_stri
     rope_kv_kernel<float><<<grid, threads, 0, stream>>>(
         (float*)q, q_stride, (const float*)k, k_stride, (const float*)v, v_stride, pos, req, freqs, v_freqs,
         (float*)k_pages, (float*)v_pages, block_table, table_width, page_size, n_pages, n_heads,
-        n_kv_heads, head_dim, status, vec, ipt, rstd, qn_w, kn_w, rstd_heads);
+        n_kv_heads, head_dim, status, vec, ipt, rstd, qn_w, kn_w, rstd_heads, magnitude, rot_pairs);
   else if (dtype == FG_BF16)
     rope_kv_kernel<__nv_bfloat16><<<grid, threads, 0, stream>>>(
         (__nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)k, k_stride, (const __nv_bfloat16*)v,
         v_stride, pos, req, freqs, v_freqs, (__nv_bfloat16*)k_pages, (__nv_bfloat16*)v_pages, block_table,
-        table_width, page_size, n_pages, n_heads, n_kv_heads, head_dim, status, vec, ipt, rstd, qn_w, kn_w, rstd_heads);
+        table_width, page_size, n_pages, n_heads, n_kv_heads, head_dim, status, vec, ipt, rstd, qn_w, kn_w, rstd_heads, magnitude, rot_pairs);
   else
     FG_CHECK_ARG(false, "fg_rope_kv_write: bad dtype %d", dtype);
   FG_CHECK_LAUNCH("fg_rope_kv_write");

@@ -63,7 +63,8 @@ class GQAAttention(Mixer):
     the keys as projected (no value projection); a query temperature that grows with the position; a
     sink per head in the softmax's denominator; a sigmoid gate per head on the output; a short causal
     convolution over time on q, k and v directly after the projection, whose last inputs are the
-    request's fixed-size state beside its pages.
+    request's fixed-size state beside its pages; chunks instead of a window; a sink with a constant score;
+    a factor on cosine and sine of the rotation (the encoding's ``magnitude``).
     """
 
     params: AttentionParams
@@ -83,7 +84,10 @@ class GQAAttention(Mixer):
         #: channels that pass the convolution: q, k and v as the kernels hold them (padded heads)
         self.conv_channels = self.q_width + 2 * self.kv_width
         #: the fused few-token kernel (projection, rotation, page write) knows none of these
-        self.plain = not (p.qk_norm or p.q_temp or p.conv or p.head_gate)
+        #: what cosine and sine are multiplied by, and the number of pairs that turn
+        self.magnitude = getattr(self.position, "magnitude", lambda: 1.0)()
+        self.rot_pairs = self._rot_dims(self.position, p.head_dim) // 2
+        self.plain = not (p.qk_norm or p.q_temp or p.conv or p.head_gate or self.magnitude != 1.0)
         if p.q_temp and p.qk_norm == "projection":
             raise ValueError("a query temperature joins the per-head factors: not with a norm over the projection")
 
@@ -131,7 +135,7 @@ class GQAAttention(Mixer):
 
     def cache_spec(self) -> Optional[CacheSpec]:
         p = self.params
-        return CacheSpec(p.n_kv_heads, self.hd, p.window, keep_first=p.keep_first if p.window else 0)
+        return CacheSpec(p.n_kv_heads, self.hd, p.window, keep_first=p.keep_first if p.window else 0, chunk=p.chunk)
 
     def state_spec(self) -> Optional[StateSpec]:
         p = self.params
@@ -195,6 +199,8 @@ class GQAAttention(Mixer):
             self.q_norm = self._rows(qn, p.n_heads, p.head_dim, p.qk_layout, qk_pos).float().contiguous()
             self.k_norm = self._rows(kn, p.n_kv_heads, p.head_dim, p.qk_layout, qk_pos).float().contiguous()
         self.sinks = tensors["sink"].float().contiguous() if p.sink else None
+        if p.sink_score is not None:
+            self.sinks = torch.full((p.n_heads,), p.sink_score, dtype=torch.float32, device=ops.device)
         self.conv_w = None
         if p.conv:
             self.conv_w = torch.cat([
@@ -223,7 +229,7 @@ class GQAAttention(Mixer):
         p = self.params
         return self.ops.attention(q, o, memory, ctx, p.n_heads, p.n_kv_heads, self.hd, p.window, self.scale,
                                   out_freqs=self.v_unfreqs, keep_first=p.keep_first, softcap=p.softcap,
-                                  sinks=self.sinks)
+                                  sinks=self.sinks, chunk=p.chunk)
 
     def forward(self, x, ctx, memory):
         p, ops = self.params, self.ops
@@ -269,7 +275,7 @@ class GQAAttention(Mixer):
             ops.rope_kv_write(
                 q, k, v, ctx.pos, ctx.req, self.freqs, memory.k_pages, memory.v_pages,
                 memory.block_table, memory.page_size, p.n_heads, p.n_kv_heads, self.hd, v_freqs=self.v_freqs,
-                qk_norm=qk_norm,
+                qk_norm=qk_norm, magnitude=self.magnitude, rot_pairs=self.rot_pairs,
             )
         o = torch.empty((t, self.q_width), dtype=x.dtype, device=x.device)
         turned = self._attend(q, o, ctx, memory)

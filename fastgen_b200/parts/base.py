@@ -53,12 +53,15 @@ class CacheSpec:
     n_pools: int = 2  # 2: keys and values; 1: one entry per token
     page_size: Optional[int] = None  # tokens per page; None: the engine's page size
     keep_first: int = 0  # with a window: a sequence's first positions that stay visible for good
+    chunk: Optional[int] = None  # a query sees only the keys of its own chunk of so many positions (from 0 on)
 
     def __post_init__(self) -> None:
         if self.n_pools not in (1, 2):
             raise ValueError(f"a cache spec asks for 1 or 2 pools, got {self.n_pools}")
         if self.page_size is not None and self.page_size <= 0:
             raise ValueError(f"page size must be positive, got {self.page_size}")
+        if self.chunk is not None and (self.chunk <= 0 or self.window is not None):
+            raise ValueError(f"a chunk is a positive number of positions and excludes a window, got {self.chunk}")
 
 
 @dataclass(frozen=True)
@@ -119,7 +122,8 @@ class Norm(Part):
 
         The default composes the steps; implementations may fuse them."""
         if isinstance(delta, ScaledSum):
-            delta = self._joined(h, delta, rows)
+            # (a summand that a norm closes is formed beside the stream)
+            delta = self._joined(h, delta, True if delta_norm is not None else rows)
         if delta is not None:
             if delta_norm is not None:
                 delta = delta_norm.forward(delta, out_dtype=torch.float32)

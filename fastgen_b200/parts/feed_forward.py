@@ -11,7 +11,7 @@ from .params import DenseMLPParams, SwiGLUParams
 
 
 class SwiGLU(FeedForward):
-    """``w2(silu(w1 x) * w3 x)`` (fastgen/forward.py:491-496).  Gate and up run
+    """``w2(act(w1 x) * w3 x)`` (fastgen/forward.py:491-496, with SiLU).  Gate and up run
     as one product against ``[w1; w3]``; the activation is computed in float32
     and rounded once."""
 
@@ -46,11 +46,11 @@ class SwiGLU(FeedForward):
         g = None
         if x.dtype == torch.bfloat16 and self.interleave:
             # a few tokens: product and gate in one kernel, the [gate | up] rows never exist
-            g = ops.linear_swiglu(x, self.w13)
+            g = ops.linear_swiglu(x, self.w13, act=self.params.act)
         if g is None:
             x13 = ops.linear(x, self.w13)
             g = torch.empty((x.shape[0], self.params.ffn_dim), dtype=x.dtype, device=x.device)
-            ops.silu_gate(x13, g, self.interleave)
+            ops.silu_gate(x13, g, self.interleave, act=self.params.act)
         return ops.linear(g, self.w2)
 
 

@@ -1,4 +1,4 @@
-"""RMSNorm, fused with the residual sum that precedes it."""
+"""Norms, fused with the residual sum that precedes them."""
 
 from __future__ import annotations
 
@@ -8,6 +8,9 @@ import torch
 
 from .base import Norm, ScaledSum, StreamUpdate, WeightSpec, register_norm
 from .params import DynamicTanhParams, LayerNormParams, PartRMSNormParams, RMSNormParams
+
+#: widest row that one kernel norms on both sides of a residual sum
+LAYER_NORM_PAIR_MAX_DIM = 8192
 
 
 class RMSNorm(Norm):
@@ -93,7 +96,7 @@ class DynamicTanh(Norm):
 
     def add_forward(self, h, delta, rows=None, delta_norm=None):
         if isinstance(delta, ScaledSum):
-            delta = self._joined(h, delta, rows)
+            delta = self._joined(h, delta, True if delta_norm is not None else rows)
         if delta is not None and delta_norm is not None and not isinstance(delta_norm, DynamicTanh):
             delta, delta_norm = delta_norm.forward(delta, out_dtype=torch.float32), None
         n = h.shape[0] if rows is None else rows.numel()
@@ -104,7 +107,12 @@ class DynamicTanh(Norm):
 
 class LayerNorm(Norm):
     """``(x - mean) / sqrt(var + eps) * w + b`` in float32; the variance is the mean of the squared
-    deviations.  Tensors ``weight`` and, with ``params.bias``, ``bias``.
+    deviations.  Tensors ``weight`` and, with ``params.bias``, ``bias``; with ``params.scale`` the
+    tensor ``scale`` multiplies the result (it is folded into the two others, in float32).
+
+    When a layer norm closes a sub-layer and another one opens the next, ``add_forward`` runs both and
+    the residual sum between them in one kernel, which also forms the sub-layer's output when that is
+    a :class:`ScaledSum`.
 
     The residual stream may be several streams ``h`` [T, S, dim] that are mixed on the way
     (``streams_forward``): the update a sub-layer left pending, the weighted sum of the streams
@@ -118,12 +126,15 @@ class LayerNorm(Norm):
         specs = [WeightSpec(self.names["weight"], (d,), ("ones",))]
         if self.params.bias:
             specs.append(WeightSpec(self.names["bias"], (d,), ("normal", 0.02)))
+        if self.params.scale:
+            specs.append(WeightSpec(self.names["scale"], (d,), ("ones",)))
         return specs
 
     def bind(self, tensors, ops) -> None:
         self.ops = ops
-        self.weight = tensors["weight"].float().contiguous()
-        self.bias = tensors["bias"].float().contiguous() if self.params.bias else None
+        scale = tensors["scale"].float() if self.params.scale else 1.0
+        self.weight = (tensors["weight"].float() * scale).contiguous()
+        self.bias = (tensors["bias"].float() * scale).contiguous() if self.params.bias else None
 
     def streams_forward(self, h, update=None, in_coef=None, rows=None, out_dtype=None):
         """``h`` [T, S, dim] (or [T, dim]): apply ``update`` (a :class:`StreamUpdate` or ``None``),
@@ -139,8 +150,15 @@ class LayerNorm(Norm):
         return self.streams_forward(x, rows=rows, out_dtype=out_dtype)
 
     def add_forward(self, h, delta, rows=None, delta_norm=None):
+        if delta is not None and isinstance(delta_norm, LayerNorm) and h.dim() == 2:
+            total = ScaledSum.of(delta)
+            if h.shape[1] <= LAYER_NORM_PAIR_MAX_DIM and total.row is None and 1 <= len(total.terms) <= 4 and len({t.dtype for t, _ in total.terms}) == 1:
+                n = h.shape[0] if rows is None else rows.numel()
+                out = torch.empty((n, h.shape[1]), dtype=self.ops.act_dtype, device=h.device)
+                return self.ops.layer_norm_pair(h, total.terms, delta_norm.weight, delta_norm.bias, delta_norm.params.eps,
+                                                self.weight, self.bias, self.params.eps, out, rows=rows)
         if isinstance(delta, ScaledSum):
-            delta = self._joined(h, delta, rows)
+            delta = self._joined(h, delta, True if delta_norm is not None else rows)
         if delta is not None and delta_norm is not None:
             delta = delta_norm.forward(delta, out_dtype=torch.float32)
         update = StreamUpdate(delta) if delta is not None else None

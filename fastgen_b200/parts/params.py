@@ -100,6 +100,9 @@ class AttentionParams:
     #: with a window: so many of a sequence's first positions stay visible to every later
     #: query, at their true positions
     keep_first: int = 0
+    #: a query sees only the keys of its own chunk: positions ``i`` and ``j <= i`` with ``i // chunk ==
+    #: j // chunk``, counted from the sequence's start (excludes a window)
+    chunk: Optional[int] = None
     #: ``"projection"``: queries and keys pass an RMS norm over their whole projection (all heads of
     #: a token at once, eps ``qk_norm_eps``, plain weights ``q_norm`` / ``k_norm`` of that size) before
     #: they are rotated; ``"head"``: an RMS norm per head, weights of ``head_dim`` numbers shared by the
@@ -119,6 +122,9 @@ class AttentionParams:
     #: the softmax's denominator also holds ``exp(sink[h])`` for query head ``h`` (tensor ``sink``): a score
     #: without a key or a value, not scaled, counted once
     sink: bool = False
+    #: a sink whose score is this number for every head (no tensor; excludes ``sink``): 0.0 adds one to the
+    #: softmax's denominator
+    sink_score: Optional[float] = None
     #: head ``h``'s output is multiplied by ``sigmoid(wg x)[h]`` before the output projection (tensor
     #: ``wg`` [heads, dim]; ``x`` is the mixer's input)
     head_gate: bool = False
@@ -157,6 +163,10 @@ class AttentionParams:
                 raise ValueError(f"head size {size} is odd: a rotation needs pairs of dimensions")
         if self.window is not None and self.window <= 0:
             raise ValueError(f"attention window must be positive, got {self.window}")
+        if self.chunk is not None and (self.chunk <= 0 or self.window is not None):
+            raise ValueError(f"a chunk is a positive number of positions and excludes a window, got {self.chunk}")
+        if self.sink and self.sink_score is not None:
+            raise ValueError("a sink's score is a tensor or a constant, not both")
         if self.keep_first < 0:
             raise ValueError(f"the number of first positions kept visible cannot be negative, got {self.keep_first}")
 
@@ -177,13 +187,24 @@ class SigmoidAttentionParams(AttentionParams):
     gate: bool = True
     distance_bias: bool = True
 
+    def __post_init__(self) -> None:
+        super().__post_init__()
+        if self.chunk is not None or self.sink or self.sink_score is not None:
+            raise ValueError("attention with sigmoid weights takes neither chunks nor sinks")
+
 
 @dataclass(frozen=True)
 class SwiGLUParams:
-    """Dense gated feed-forward ``w2(silu(w1 x) * w3 x)`` (forward.py:491-496)."""
+    """Dense gated feed-forward ``w2(act(w1 x) * w3 x)`` (forward.py:491-496, with SiLU); ``act`` is
+    ``"silu"`` or ``"relu"``."""
 
     dim: int
     ffn_dim: int
+    act: str = "silu"
+
+    def __post_init__(self) -> None:
+        if self.act not in ("silu", "relu"):
+            raise ValueError(f"unknown activation of a gate {self.act!r}")
 
 
 @dataclass(frozen=True)
@@ -259,11 +280,13 @@ class BigramHashParams:
 @dataclass(frozen=True)
 class LayerNormParams:
     """``(x - mean) / sqrt(var + eps) * w + b`` with the variance the mean of the squared
-    deviations; ``bias`` says whether the norm has a ``b``."""
+    deviations; ``bias`` says whether the norm has a ``b``.  With ``scale`` the result is also multiplied,
+    element by element, by the tensor ``scale`` (a layer scale behind the norm that closes a sub-layer)."""
 
     dim: int
     eps: float
     bias: bool = True
+    scale: bool = False
 
 
 @dataclass(frozen=True)
@@ -314,6 +337,25 @@ class Mamba2Params:
 
 
 @dataclass(frozen=True)
+class SelectiveScanParams:
+    """The selective state-space mixer in the Mamba-1 form: ``inner`` channels with a state of ``state``
+    numbers each, step sizes through a low-rank map of inner size ``dt_rank``, a causal convolution of
+    ``conv`` taps (with bias) per channel."""
+
+    dim: int
+    inner: int
+    state: int
+    dt_rank: int
+    conv: int
+
+    def __post_init__(self) -> None:
+        if not 1 <= self.conv <= 8:
+            raise ValueError(f"the convolution takes 1 to 8 taps, got {self.conv}")
+        if not 1 <= self.state <= 256:
+            raise ValueError(f"a channel's state takes 1 to 256 numbers, got {self.state}")
+
+
+@dataclass(frozen=True)
 class LatentAttentionParams:
     """Causal softmax attention whose keys and values are linear maps of a cached latent.
 
@@ -358,7 +400,11 @@ class GatedDeltaParams:
     queries and keys have ``n_kv_heads`` heads (head ``h`` uses ``h // (n_heads / n_kv_heads)``).
     q, k and v pass a causal convolution of ``conv`` taps per channel and SiLU.  The decay per head
     and key channel and the gate of the output come through two low-rank maps whose inner sizes are
-    ``decay_rank`` and ``gate_rank`` (``None``: whatever the checkpoint's tensors have)."""
+    ``decay_rank`` and ``gate_rank`` (``None``: whatever the checkpoint's tensors have).
+
+    ``head_decay``: one decay per head, from one projection (tensor ``wa`` [heads, dim]).  ``full_gate``:
+    the output's gate is one projection (tensor ``wg`` [heads * v_head_dim, dim]).  ``gate_act``: what the
+    gate passes, ``"sigmoid"`` or ``"silu"``."""
 
     dim: int
     n_heads: int
@@ -369,8 +415,13 @@ class GatedDeltaParams:
     eps: float
     decay_rank: Optional[int] = None
     gate_rank: Optional[int] = None
+    head_decay: bool = False
+    full_gate: bool = False
+    gate_act: str = "sigmoid"
 
     def __post_init__(self) -> None:
+        if self.gate_act not in ("sigmoid", "silu"):
+            raise ValueError(f"unknown gate {self.gate_act!r}")
         if self.n_heads % self.n_kv_heads:
             raise ValueError(f"{self.n_heads} heads cannot share {self.n_kv_heads} query/key heads")
         if not 1 <= self.conv <= 8:
@@ -434,6 +485,8 @@ class RoutedExpertsParams:
     #: the router's logits have a bias (tensor ``router_bias`` [experts]) that counts in the choice and in
     #: the weights
     router_bias: bool = False
+    #: an expert's weight multiplies its input instead of its output: ``sum_e expert_e(weight_e x)``
+    weigh_input: bool = False
 
     def __post_init__(self) -> None:
         if not 1 <= self.top <= self.n_experts:

@@ -26,7 +26,9 @@ class RoutedExperts(FeedForward):
     factor on the weights; a bias of the router's logits; experts without a gate, ``w2_e(act(w3_e x))``; a
     shared feed-forward that every token passes and whose output is added (the result is then a sum that
     the next norm's kernel forms), or multiplied by the sigmoid of one number per token and added (the
-    number is one more row of the router's product, and the kernel that sums the experts adds it).
+    number is one more row of the router's product, and the kernel that sums the experts adds it); weights
+    that multiply the experts' inputs instead of their outputs (the first products' kernels multiply their
+    sums by them, which is the same).
     """
 
     params: RoutedExpertsParams
@@ -116,7 +118,8 @@ class RoutedExperts(FeedForward):
         shared = self.shared.forward(x, ctx) if self.shared is not None else None
         gated = gate is not None  # (then the experts' sum takes the shared output in)
         out = ops.moe_experts(x, ids, weights, self.w1, self.w3, self.w2, self.w13, act=None if self.gated else p.act,
-                              shared=shared if gated else None, shared_gate=gate)
+                              shared=shared if gated else None, shared_gate=gate,
+                              weigh_input=p.weigh_input)
         if shared is None or gated:
             return out
         return ScaledSum([(out, 1.0), (shared, 1.0)])
