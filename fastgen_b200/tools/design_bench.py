@@ -1,6 +1,6 @@
 """Throughput of one design beside another at equal size, step by step and kernel by kernel.
 
-``bench.py --design sinorax|zeladra|tanupel|palulorn|kuvusun`` runs this: prefill and decode throughput of a model of that
+``bench.py --design sinorax|zeladra|tanupel|palulorn|kuvusun|pegurax`` runs this: prefill and decode throughput of a model of that
 design at a few sizes that resemble a real model's layers (random weights), beside a Llama-shaped model of
 the same width, heads, head size, number of layers and number of parameters a layer, and the
 time of each kernel family of the two designs at those sizes with its fraction of the roofline
@@ -150,6 +150,26 @@ def kuvusun_config(width, layers, heads, kv, head_dim, ffn, vocab, window=None, 
     return dict(architecture="Kuvusun", vocab=vocab, width=width, norm=dict(eps=1e-5, groups=8), layers=out)
 
 
+def pegurax_config(width, layers, heads, kv, head_dim, ffn, vocab, chunk=1024, experts=8, top=2) -> dict:
+    """A pair of mixers (attention inside chunks with half the heads beside a gated delta rule with the other
+    half) and the selective scan (``width`` channels of 16 numbers, about the parameters of the Llama shape's
+    attention), in turn; the feed-forwards are dense and routed in turn, as Tanupel's above."""
+    left = dict(heads=heads // 2, kv_heads=max(1, kv // 2), dim=head_dim, vdim=head_dim, scale=head_dim ** -0.5, mask=dict(size=chunk),
+                rot=dict(dims=head_dim, base=500000.0, scaling=dict(factor=8.0, original=8192, fast=32.0, slow=1.0)))
+    right = dict(heads=heads // 2, kv_heads=max(1, kv // 2), dim=head_dim, vdim=head_dim, conv=4)
+    scan = dict(inner=width, state=16, dt_rank=width // 16, conv=4)
+    dense = dict(kind="dense", ff=ffn)
+    routed = dict(kind="moe", expert=dict(ff=ffn // experts), router=dict(experts=experts, top=top))
+    out = []
+    for i in range(layers):
+        mlp = dict(dense if (i // 2) % 2 == 0 else routed)
+        if i % 2 == 0:
+            out.append(dict(type="parallel", mixer=dict(left=left, right=right, left_scale=0.8, right_scale=0.5), mlp=mlp))
+        else:
+            out.append(dict(type="mamba1", mixer=dict(scan), mlp=mlp))
+    return dict(architecture="Pegurax", vocab=vocab, width=width, norm=dict(eps=1e-5), embedding=dict(scale=1.0), layers=out)
+
+
 class Timer:
     """CUDA-event times of single launches, each after a write larger than L2."""
 
@@ -281,7 +301,8 @@ def model_throughput(cfg, device) -> Dict[str, float]:
     return out
 
 
-def _attention_times(cfg, device, timer: Timer, layer: int, flops_window, heads, kv, head_dim, pick=None) -> Dict[str, float]:
+def _attention_times(cfg, device, timer: Timer, layer: int, flops_window, heads, kv, head_dim, pick=None,
+                     chunk=None) -> Dict[str, float]:
     """The attention launches of one layer alone: a 2,048-token prompt, and 8 single tokens at
     position 2,048, with what the mixer adds around them (turning the outputs back)."""
     from ..engine import StepEntry
@@ -309,7 +330,7 @@ def _attention_times(cfg, device, timer: Timer, layer: int, flops_window, heads,
     o = torch.empty_like(q)
     us = timer.us(lambda: mixer._attend(q, o, ctx, memory))
     w = flops_window or PREFILL_TOKENS
-    keys = sum(min(i + 1, w) for i in range(PREFILL_TOKENS))
+    keys = sum(i % chunk + 1 if chunk else min(i + 1, w) for i in range(PREFILL_TOKENS))
     out["prefill_us"] = round(us, 1)
     out["prefill_tflops"] = round(4 * head_dim * heads * keys / (us * 1e-6) / 1e12, 1)
     if getattr(mixer, "v_unfreqs", None) is not None:
@@ -701,6 +722,169 @@ def tanupel_kernel_table(size, device, peaks) -> Dict[str, dict]:
     return table
 
 
+def pegurax_kernel_table(size, device, peaks) -> Dict[str, dict]:
+    """The kernels of the Pegurax design alone at one size, each beside the like kernel of the closest model
+    (Tanupel's delta rule and routed experts, Zeladra's state-space recurrence and layer norm, the Llama shape's
+    attention with a window and its feed-forward): microseconds and the fraction of the roofline.  Rows of few
+    tokens are timed as captured launches."""
+    from ..csrc.ops import Ops
+    from ..engine.step import StepContext
+
+    width, _layers, heads, kv, head_dim, ffn, vocab, window = size
+    ops = Ops(torch.bfloat16, device)
+    timer = Timer(device)
+    gen = torch.Generator().manual_seed(SEED)
+    hbm, tensor = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    table: Dict[str, dict] = {}
+
+    def bw(name, us, nbytes):
+        table[name] = dict(us=round(us, 1), gbs=round(nbytes / (us * 1e-6) / 1e9, 1), hbm_frac=round(nbytes / (us * 1e-6) / hbm, 3))
+
+    def rand(*shape, dtype=torch.bfloat16):
+        return torch.randn(*shape, generator=gen).to(device, dtype)
+
+    def context(t, n_seqs):
+        ctx = StepContext(device)
+        per = t // n_seqs
+        ctx.req = torch.arange(n_seqs, dtype=torch.int32, device=device).repeat_interleave(per)
+        ctx.pos = torch.arange(per, dtype=torch.int32, device=device).repeat(n_seqs)
+        ctx.seq_slot = torch.arange(n_seqs, dtype=torch.int32, device=device)
+        ctx.seq_start = torch.arange(0, t + 1, per, dtype=torch.int32, device=device)
+        ctx.n_tokens, ctx.n_seqs = t, n_seqs
+        return ctx
+
+    few = lambda t: t == DECODE_BATCH
+    cfg = pegurax_config(*size)
+    right = cfg["layers"][0]["mixer"]["right"]
+    for t in (PREFILL_TOKENS, DECODE_BATCH):
+        h = rand(t, width, dtype=torch.float32)
+        out = torch.empty(t, width, dtype=torch.bfloat16, device=device)
+        w1, w2 = rand(width, dtype=torch.float32), rand(width, dtype=torch.float32)
+        a, b = rand(t, width), rand(t, width)
+        for n, terms in ((1, [(a, 1.0)]), (2, [(a, 0.8), (b, 0.5)])):
+            bw(f"norm+sum t={t}: two layer norms around a sum of {n}", timer.us(lambda: ops.layer_norm_pair(
+                h, terms, w1, None, 1e-5, w2, None, 1e-5, out), graph=few(t)), t * width * (4 + 4 + 2 * n + 2))
+        from ..parts.base import StreamUpdate
+        bw(f"norm+sum t={t}: layer norm (sum, norm; zeladra's kernel)", timer.us(lambda: ops.stream_norm(
+            h, w1, None, 1e-5, out, update=StreamUpdate(a)), graph=few(t)), t * width * (4 + 4 + 2 + 2))
+        wb = rand(width)
+        bw(f"norm+sum t={t}: rmsnorm (sum, norm; llama)", timer.us(lambda: ops.rmsnorm(h, wb, 1e-5, out=out, delta=a), graph=few(t)),
+           t * width * (4 + 4 + 2 + 2))
+
+    # the gated delta rule with one decay a head beside the one with a decay a key channel
+    H, G, d, dv, taps = right["heads"], right["kv_heads"], right["dim"], right["vdim"], right["conv"]
+    channels = 2 * G * d + H * dv
+    state = torch.zeros(DECODE_BATCH, H * dv * d + (taps - 1) * channels, dtype=torch.float32, device=device)
+    conv_w = rand(channels, taps, dtype=torch.float32)
+    dt_bias, a_log, norm_w = rand(H * d, dtype=torch.float32), rand(H, dtype=torch.float32), rand(dv, dtype=torch.float32)
+    for t, n_seqs in ((PREFILL_TOKENS, 1), (DECODE_BATCH, DECODE_BATCH)):
+        proj, a, b, z = rand(t, channels), rand(t, H * d), rand(t, H), rand(t, H * dv)
+        ctx = context(t, n_seqs)
+        qkv = ops.conv_silu(proj, 0, channels, conv_w, state, H * dv * d, taps, ctx)
+        state_bytes = n_seqs * H * dv * d * 8
+        for what, head in (("a decay a head", True), ("a decay a key channel; tanupel", False)):
+            aa, bias = (a[:, :H].contiguous(), dt_bias[:H].contiguous()) if head else (a, dt_bias)
+            bw(f"delta rule t={t}: recurrence, {what} ({n_seqs} sequences, {H} heads, state {d} x {dv})", timer.us(lambda: ops.delta_scan(
+                qkv, aa, b, bias, a_log, state, ctx, H, G, d, dv, head_decay=head), graph=few(t)),
+               t * (channels * 4 + aa.shape[1] * 2 + H * dv * 4) + state_bytes)
+            state.zero_()
+        y = rand(t, H * dv, dtype=torch.float32)
+        for act in ("silu", "sigmoid"):
+            bw(f"delta rule t={t}: norm per head + {act} gate", timer.us(lambda: ops.head_norm_gate(y, z, norm_w, H, dv, 1e-5, ctx, act=act),
+                                                                     graph=few(t)), t * H * dv * (4 + 2 + 2))
+
+    # the selective scan beside Zeladra's state-space recurrence (as many state numbers, and at this width)
+    scan = cfg["layers"][1]["mixer"]
+    N = scan["state"]
+    for inner in (scan["inner"], 2 * width):
+        sstate = torch.zeros(DECODE_BATCH, inner * N + 3 * inner, dtype=torch.float32, device=device)
+        vec = [rand(inner, dtype=torch.float32) for _ in range(2)]
+        rates = -torch.exp(rand(inner, N, dtype=torch.float32))
+        cw, cb = rand(inner, 4, dtype=torch.float32), rand(inner, dtype=torch.float32)
+        for t, n_seqs in ((PREFILL_TOKENS, 1), (DECODE_BATCH, DECODE_BATCH)):
+            ctx = context(t, n_seqs)
+            proj, dt, low = rand(t, 2 * inner), rand(t, inner), rand(t, 2 * N)
+            bw(f"selective scan t={t}: convolution + SiLU ({inner} channels)", timer.us(lambda: ops.time_conv(
+                proj, 0, inner, cw, cb, sstate, inner * N, 4, ctx, act="silu", out_dtype=torch.bfloat16), graph=few(t)), t * inner * 4)
+            u = ops.time_conv(proj, 0, inner, cw, cb, sstate, inner * N, 4, ctx, act="silu", out_dtype=torch.bfloat16)
+            bw(f"selective scan t={t}: recurrence and gate ({n_seqs} sequences, {inner} channels of {N})", timer.us(lambda: ops.selective_scan(
+                u, dt, low, 0, proj[:, inner:], vec[0], rates, vec[1], sstate, ctx, N), graph=few(t)),
+               t * (inner * 8 + 4 * N) + n_seqs * inner * N * 8)
+            sstate.zero_()
+    ssm = zeladra_config(*size)["layers"][1]["mixer"]
+    sH, P, sN, sG, staps = ssm["heads"], ssm["vdim"], ssm["state"], ssm["groups"], ssm["conv"]
+    inner, sch = sH * P, sH * P + 2 * sG * sN
+    cols = 2 * inner + 2 * sG * sN + sH
+    sstate = torch.zeros(DECODE_BATCH, sH * sN * P + (staps - 1) * sch, dtype=torch.float32, device=device)
+    sconv_w, sconv_b = rand(sch, staps, dtype=torch.float32), rand(sch, dtype=torch.float32)
+    vec, nw = [rand(sH, dtype=torch.float32) for _ in range(3)], rand(inner, dtype=torch.float32)
+    for t, n_seqs in ((PREFILL_TOKENS, 1), (DECODE_BATCH, DECODE_BATCH)):
+        proj = rand(t, cols)
+        ctx = context(t, n_seqs)
+        bw(f"state-space (zeladra) t={t}: convolution + SiLU ({sch} channels)", timer.us(lambda: ops.mamba2_conv(
+            proj, inner, sch, sconv_w, sconv_b, sstate, sH * sN * P, staps, ctx), graph=few(t)), t * sch * 6)
+        xbc = ops.mamba2_conv(proj, inner, sch, sconv_w, sconv_b, sstate, sH * sN * P, staps, ctx)
+
+        def recurrence():
+            y = ops.mamba2_scan(xbc, proj, inner + sch, *vec, sstate, ctx, sH, sG, sN, P)
+            return ops.gated_part_norm(y, proj[:, :inner], nw, 8, 1e-5, ctx)
+        bw(f"state-space (zeladra) t={t}: recurrence, gate and norm ({n_seqs} sequences, {sH} heads, state {sN} x {P})",
+           timer.us(recurrence, graph=few(t)), t * (sch * 4 + inner * (4 + 4 + 2 + 2)) + n_seqs * sH * sN * P * 8)
+        sstate.zero_()
+
+    # routed experts: weights on the inputs beside weights on the outputs
+    mlp = cfg["layers"][2]["mlp"]
+    E, top, f = mlp["router"]["experts"], mlp["router"]["top"], mlp["expert"]["ff"]
+    w13, w2 = rand(E, 2 * f, width), rand(E, width, f)
+    w1, w3 = w13[:, :f], w13[:, f:]
+    router = rand(E, width, dtype=torch.float32)
+    wd13, wd = rand(2 * ffn, width), rand(width, ffn)
+    for t in (PREFILL_TOKENS, DECODE_BATCH):
+        x = rand(t, width)
+        ctx = context(t, 1)
+        logits = ops.moe_logits(x, router)
+        for score, weigh in (("sigmoid", True), ("softmax", False)):
+            ids, weights = ops.moe_route(logits, None, top, ctx, score=score)
+            us = timer.us(lambda: ops.moe_experts(x, ids, weights, w1, w3, w2, w13, weigh_input=weigh), graph=few(t))
+            touched = min(E, t * top)
+            table[f"routed experts t={t}: {top} of {E} experts of {f} rows, weights on the {'inputs' if weigh else 'outputs; tanupel'}"] = dict(
+                choice_us=round(timer.us(lambda: ops.moe_route(logits, None, top, ctx, score=score), graph=few(t)), 1),
+                experts_us=round(us, 1), experts_tensor_frac=round(6 * t * top * f * width / (us * 1e-6) / tensor, 3),
+                experts_hbm_frac=round(touched * 3 * f * width * 2 / (us * 1e-6) / hbm, 3))
+        for act in ("relu", "silu"):
+            def dense():
+                g = ops.linear_swiglu(x, wd13, act=act)
+                if g is None:
+                    g = torch.empty(t, ffn, dtype=torch.bfloat16, device=device)
+                    ops.silu_gate(ops.linear(x, wd13), g, 8, act=act)
+                return ops.linear(g, wd)
+            us = timer.us(dense, graph=few(t))
+            table[f"dense gated feed-forward t={t}: {ffn} rows, {act}{' (llama)' if act == 'silu' else ''}"] = dict(
+                us=round(us, 1), tensor_frac=round(6 * t * ffn * width / (us * 1e-6) / tensor, 3),
+                hbm_frac=round(3 * ffn * width * 2 / (us * 1e-6) / hbm, 3))
+
+    small = (width, 2, heads, kv, head_dim, ffn, 1024)
+    pz = pegurax_config(*small, window)
+    left = pz["layers"][0]["mixer"]["left"]
+    table[f"attention softmax, chunks and sink (pegurax pair's left half, chunk {window})"] = _attention_times(
+        pz, device, timer, 0, window, left["heads"], left["kv_heads"], head_dim, pick=lambda m: m.left, chunk=window)
+    half = (width, 2, heads // 2, max(1, kv // 2), head_dim, ffn, 1024)
+    table[f"attention softmax (llama, half the heads, window {window})"] = _attention_times(
+        llama_config(*half, window=window), device, timer, 0, window, heads // 2, max(1, kv // 2), head_dim)
+    for name, row in table.items():
+        if "prefill_tflops" in row:
+            row["prefill_tensor_frac"] = round(row["prefill_tflops"] * 1e12 / tensor, 3)
+            row["decode_hbm_frac"] = round(row["decode_gbs"] * 1e9 / hbm, 3)
+    tz = tanupel_config(*small)
+    table["mixer pair (pegurax; whole mixer)"] = _mixer_times(pz, device, timer, 0)
+    table["mixer pair (tanupel; whole mixer)"] = _mixer_times(tz, device, timer, 0)
+    table["mixer pair's right half alone (pegurax delta rule; whole mixer)"] = _mixer_times(pz, device, timer, 0, pick=lambda b: b.mixer.right)
+    table["mixer pair's right half alone (tanupel delta rule; whole mixer)"] = _mixer_times(tz, device, timer, 0, pick=lambda b: b.mixer.right)
+    table["mixer selective scan (pegurax; whole mixer)"] = _mixer_times(pz, device, timer, 1)
+    table["mixer state-space (zeladra; whole mixer)"] = _mixer_times(zeladra_config(*small, window), device, timer, 1)
+    return table
+
+
 def palulorn_kernel_table(size, device, peaks) -> Dict[str, dict]:
     """The kernels of the Palulorn design alone at one size, each beside the like kernel of the closest
     model where there is one (Tanupel's delta rule for the matrix memory, its routed experts, the Llama
@@ -987,6 +1171,23 @@ def kuvusun_kernel_table(size, device, peaks) -> Dict[str, dict]:
 def run(sizes: List[str], peaks: dict, kernels: bool = True, design: str = "sinorax") -> dict:
     device = torch.device("cuda:0")
     torch.cuda.set_device(device)
+    if design == "pegurax":
+        out = {"metric": "prefill and decode tokens/s of Pegurax beside Tanupel and a Llama-shaped model of equal size (bf16, random weights)",
+               "unit": "tokens/s", "dtype": "bf16", "data": "synthetic (random weights, uniform random token ids)",
+               "config": dict(prefill_tokens=PREFILL_TOKENS, decode_batch=DECODE_BATCH, decode_context=DECODE_CONTEXT, page=PAGE,
+                              l2="flushed before every timed kernel; model steps stream all weights"),
+               "peaks": peaks, "sizes": {}}
+        for name in sizes:
+            size = SIZES[name]
+            entry = dict(width=size[0], layers=size[1], heads=size[2], kv_heads=size[3], head_dim=size[4], swiglu_ffn=size[5],
+                         vocab=size[6], chunk=size[7], experts=8, top=2, expert_ffn=size[5] // 8, scan_inner=size[0], scan_state=16)
+            entry["pegurax"] = model_throughput(pegurax_config(*size), device)
+            entry["tanupel"] = model_throughput(tanupel_config(*size), device)
+            entry["llama"] = model_throughput(llama_config(*size[:7]), device)
+            if kernels:
+                entry["kernels"] = pegurax_kernel_table(size, device, peaks)
+            out["sizes"][name] = entry
+        return out
     if design == "kuvusun":
         out = {"metric": "prefill and decode tokens/s of Kuvusun beside Zeladra (latent layers only) and a Llama-shaped model of equal size (bf16, random weights)",
                "unit": "tokens/s", "dtype": "bf16", "data": "synthetic (random weights, uniform random token ids)",

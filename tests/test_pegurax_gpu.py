@@ -169,10 +169,12 @@ def plain_logits(folder, tokens):
 
 
 # The bfloat16 rule of this design's models: a row of logits may differ from the plain one by T_L2 of the
-# row's l2 norm and, in its worst entry, by T_MAX of the row's largest logit.  A sub-layer's output passes a
-# norm before it joins the stream, so a rounding of a small output counts as much as one of a large output.
-# float32 rows are held to ``helpers.check_row``'s 1e-4.
-T_L2, T_MAX = 0.045, 0.055
+# row's l2 norm and, in its worst entry, by T_MAX of the row's largest logit, and a request's rows by T_MEAN of
+# their l2 norms on average.  A sub-layer's output passes a norm before it joins the stream, and so does the
+# delta rule's read-out, so where one of them happens to be small its roundings grow: the plain implementation
+# itself, with the inputs and results of its products rounded to bfloat16, is off by 0.01 of a row's norm at the
+# median and by up to 0.08 at its worst rows.  float32 rows are held to ``helpers.check_row``'s 1e-4.
+T_L2, T_MAX, T_MEAN = 0.16, 0.16, 0.025
 
 
 def check_row(row, ref, dtype, what):
@@ -182,14 +184,16 @@ def check_row(row, ref, dtype, what):
     mx = float(np.abs(row - ref).max()) / max(float(np.abs(ref).max()), 1e-30)
     assert l2 <= T_L2, f"{what}: l2 error {l2:.4f} of the row's norm (allowed {T_L2})"
     assert mx <= T_MAX, f"{what}: worst entry off by {mx:.4f} of the largest logit (allowed {T_MAX})"
+    return l2
 
 
 def compare(folder, requests, got, dtype):
     for rid, toks in requests.items():
         ref = plain_logits(folder, toks)
         assert set(got[rid]) == set(range(len(toks))), f"{rid}: positions missing"
-        for p, row in got[rid].items():
-            check_row(row, ref[p], dtype, f"{rid} pos {p}")
+        errors = [check_row(row, ref[p], dtype, f"{rid} pos {p}") for p, row in got[rid].items()]
+        if dtype == torch.bfloat16 and len(errors) >= 8:
+            assert np.mean(errors) <= T_MEAN, f"{rid}: l2 error {np.mean(errors):.4f} on average (allowed {T_MEAN})"
 
 
 def _requests(vocab, lengths, seed):
@@ -565,7 +569,7 @@ def test_keys_at_both_sides_of_a_chunks_edge(dtype, d, chunk, page):
     alone.  A chunk that is one place off, or counted from a portion's start, gives other outputs."""
     heads, n = 2, 3 * chunk + 5
     g = torch.Generator().manual_seed(chunk + d)
-    m = _attn(heads, 1, d, d, 2.0, chunk, 8, 1e4, (4.0, 4096, 32.0, 1.0))
+    m = _attn(heads, 1, d, d, 12.0 / d, chunk, 8, 1e4, (4.0, 4096, 32.0, 1.0))
 
     def tweak(w):
         for h in range(heads):
@@ -605,7 +609,7 @@ def test_far_key_inside_its_chunk(dtype, d):
     the first query of the next chunk does not: in a prompt and decoded alone, the key on the first of many pages."""
     heads, chunk, n = 2, 400, 420
     g = torch.Generator().manual_seed(21)
-    m = _attn(heads, 1, d, d, 3.0, chunk, 8, 1e4, (4.0, 4096, 32.0, 1.0))
+    m = _attn(heads, 1, d, d, 12.0 / d, chunk, 8, 1e4, (4.0, 4096, 32.0, 1.0))
 
     def tweak(w):
         for h in range(heads):
@@ -642,13 +646,13 @@ def test_the_constant_sink_joins_the_denominator_once(dtype, d):
     """Scores far below zero: almost all of the weight is the sink's, so the output is nearly zero; scores around
     zero at the first tokens of a chunk: the sink takes half, a third, a quarter.  Without it the outputs are
     several times as large; in a prompt (also one whose keys are worked on in several stretches) and decoded."""
-    m = _attn(2, 1, d, d, 0.05, 40, 8, 1e4)
+    m = _attn(2, 1, d, d, 0.5 / d, 40, 8, 1e4)
     g = torch.Generator().manual_seed(3)
     for how in ("zero", "low"):
         def tweak(w):
             w["mix.q"][:] = 0
             w["mix.k"][:] = 0
-            if how == "low":  # every score is -|.|: about -9
+            if how == "low":  # every score is -8
                 w["mix.q"][d - 1 :: d, 0] = 1.0
                 w["mix.k"][d - 1 :: d, 0] = -1.0
                 w["mix.q.norm"][:] = 4.0
@@ -1127,3 +1131,101 @@ def test_greedy_generation_through_the_entry_point(tmp_path, dtype, name):
                 logits = pp.forward(cfg, w, seq)[-1]
                 assert float(logits[tok]) >= float(logits.max()) - 0.03 * float(logits.abs().max())
                 seq.append(tok)
+
+
+# ---------------------------------------------------------------------------------
+# the rule itself, and configurations drawn at random
+# ---------------------------------------------------------------------------------
+def _edit(layers, kind, change):
+    for layer in layers:
+        if layer["type"] == kind:
+            change(layer["mixer"])
+
+
+def test_faults_break_the_bfloat16_rule(tmp_path):
+    """Negative controls, planted in the plain implementation: a chunk one place longer, a missing magnitude, a
+    frequency law without its ramp, a value head's scale, an expert's weight left out, a lost skip, a decay that is
+    a tenth off.  Each puts rows far outside what the bfloat16 comparison allows."""
+    d = model_dir(tmp_path, "pa", torch.bfloat16)
+    cfg, w = pp.read_model(d)
+    tokens = H.random_tokens(cfg["vocab"], 100, 7)
+    ref = pp.forward(cfg, w, tokens)
+
+    def off(config=cfg, tensors=w):
+        got = pp.forward(config, tensors, tokens)
+        return float(((got - ref).norm(dim=-1) / ref.norm(dim=-1)).mean())
+
+    def changed(change):
+        c = copy.deepcopy(cfg)
+        change(c["layers"])
+        return c
+    left = lambda f: (lambda layers: _edit(layers, "parallel", lambda m: f(m["left"])))
+    faults = {
+        "chunk": off(changed(left(lambda m: m["mask"].update(size=m["mask"]["size"] + 1)))),
+        "no chunks": off(changed(left(lambda m: m.pop("mask")))),
+        "no scaling": off(changed(left(lambda m: m["rot"].pop("scaling")))),
+        "ramp": off(changed(left(lambda m: m["rot"]["scaling"].update(fast=1e6, slow=1e-6)))),
+        "score scale": off(changed(left(lambda m: m.update(scale=m["scale"] * 1.2)))),
+        "left scale": off(changed(lambda layers: _edit(layers, "parallel", lambda m: m.update(left_scale=1.0)))),
+        "skip": off(tensors={k: torch.zeros_like(t) if k.endswith("mix.D") else t for k, t in w.items()}),
+        "delta decay": off(tensors={k: t + 0.3 if k.endswith("right.A_log") else t for k, t in w.items()}),
+        "scan decay": off(tensors={k: t + 1.0 if k.endswith("mix.A_log") and "right" not in k else t for k, t in w.items()}),
+        "step bias": off(tensors={k: t + 0.5 if k.endswith("dt.b") else t for k, t in w.items()}),
+        "layer scale": off(tensors={k: torch.ones_like(t) if k.endswith("ls1") else t for k, t in w.items()}),
+    }
+    assert all(v > T_MEAN for v in faults.values()), faults
+
+
+def _random_config(seed):
+    import random
+
+    r = random.Random(seed)
+    width = r.choice([40, 64, 72, 96, 120])
+
+    def attn():
+        kv = r.choice([1, 2, 3])
+        d = r.choice([8, 16, 20, 32, 48, 64, 96, 128])
+        turned = r.choice([d, d // 2, 2, None])
+        sc = r.choice([None, (r.uniform(1.5, 40), r.choice([32, 64, 512]), r.choice([4.0, 32.0]), r.choice([0.5, 1.0]))])
+        return _attn(kv * r.choice([1, 2, 4]), kv, d, r.choice([d, 8, 24, 64]), r.uniform(0.5, 2.0) * d ** -0.5,
+                     r.choice([None, 3, 16, 31, 64, 97]), turned // 2 * 2 if turned else None, r.choice([50.0, 1e4, 1e6]), sc)
+
+    def delta():
+        kv = r.choice([1, 2, 3])
+        return _delta(kv * r.choice([1, 2, 3]), kv, r.choice([8, 24, 32, 40, 64, 130]), r.choice([6, 16, 40, 64]), r.choice([1, 2, 4, 5]))
+
+    def mlp():
+        if r.random() < 0.15:
+            return None
+        if r.random() < 0.3:
+            return _dense(r.choice([20, 64, 104]))
+        e = r.choice([1, 2, 5, 8, 16])
+        return _moe(e, r.choice([1, 2, e]) if e > 1 else 1, r.choice([8, 20, 48]))
+    layers = []
+    for _ in range(r.choice([1, 2, 3])):
+        if r.random() < 0.5:
+            layer = _pair(attn(), delta(), r.uniform(0.3, 1.5), r.uniform(0.3, 1.5))
+        else:
+            layer = _mamba(r.choice([24, 50, 80, 128]), r.choice([1, 4, 16, 20, 32, 64, 100]), r.choice([1, 3, 8, 11]), r.choice([1, 2, 4, 7]))
+        layers.append(dict(layer, mlp=mlp()))
+    return dict(architecture="Pegurax", vocab=r.choice([50, 131, 256]), width=width, norm=dict(eps=r.choice([1e-6, 1e-5, 1e-3])),
+                embedding=dict(scale=r.uniform(0.5, 6.0)), layers=layers)
+
+
+@pytest.mark.gpu
+@DTYPES
+@pytest.mark.parametrize("seed", range(100, 116))
+def test_configurations_drawn_at_random(tmp_path, dtype, seed):
+    """One to three layers of sizes drawn at random, mixed batches with pages and slots that are used again."""
+    cfg = _random_config(seed)
+    name = f"random{seed}"
+    CONFIGS[name] = (cfg, seed)
+    try:
+        d = model_dir(tmp_path, name, dtype)
+        requests = _requests(cfg["vocab"], [60, 17, 1, 110, 33, 2], seed)
+        steps = H.plan_mixed(requests, seed=seed)
+        page = (4, 8, 16, 64)[seed % 4]
+        outputs, engine = H.run_engine(d, dtype, steps, page, H.max_live_tokens(steps, page) + page)
+        compare(d, requests, H.collect(steps, outputs), dtype)
+    finally:
+        del CONFIGS[name]
