@@ -725,8 +725,8 @@ def tanupel_kernel_table(size, device, peaks) -> Dict[str, dict]:
 def pegurax_kernel_table(size, device, peaks) -> Dict[str, dict]:
     """The kernels of the Pegurax design alone at one size, each beside the like kernel of the closest model
     (Tanupel's delta rule and routed experts, Zeladra's state-space recurrence and layer norm, the Llama shape's
-    attention with a window and its feed-forward): microseconds and the fraction of the roofline.  Rows of few
-    tokens are timed as captured launches."""
+    attention with a window and its feed-forward): microseconds and the fraction of the roofline.  Everything but the
+    attention and whole-mixer rows is timed as captured launches (device time)."""
     from ..csrc.ops import Ops
     from ..engine.step import StepContext
 
@@ -753,7 +753,6 @@ def pegurax_kernel_table(size, device, peaks) -> Dict[str, dict]:
         ctx.n_tokens, ctx.n_seqs = t, n_seqs
         return ctx
 
-    few = lambda t: t == DECODE_BATCH
     cfg = pegurax_config(*size)
     right = cfg["layers"][0]["mixer"]["right"]
     for t in (PREFILL_TOKENS, DECODE_BATCH):
@@ -763,12 +762,12 @@ def pegurax_kernel_table(size, device, peaks) -> Dict[str, dict]:
         a, b = rand(t, width), rand(t, width)
         for n, terms in ((1, [(a, 1.0)]), (2, [(a, 0.8), (b, 0.5)])):
             bw(f"norm+sum t={t}: two layer norms around a sum of {n}", timer.us(lambda: ops.layer_norm_pair(
-                h, terms, w1, None, 1e-5, w2, None, 1e-5, out), graph=few(t)), t * width * (4 + 4 + 2 * n + 2))
+                h, terms, w1, None, 1e-5, w2, None, 1e-5, out), graph=True), t * width * (4 + 4 + 2 * n + 2))
         from ..parts.base import StreamUpdate
         bw(f"norm+sum t={t}: layer norm (sum, norm; zeladra's kernel)", timer.us(lambda: ops.stream_norm(
-            h, w1, None, 1e-5, out, update=StreamUpdate(a)), graph=few(t)), t * width * (4 + 4 + 2 + 2))
+            h, w1, None, 1e-5, out, update=StreamUpdate(a)), graph=True), t * width * (4 + 4 + 2 + 2))
         wb = rand(width)
-        bw(f"norm+sum t={t}: rmsnorm (sum, norm; llama)", timer.us(lambda: ops.rmsnorm(h, wb, 1e-5, out=out, delta=a), graph=few(t)),
+        bw(f"norm+sum t={t}: rmsnorm (sum, norm; llama)", timer.us(lambda: ops.rmsnorm(h, wb, 1e-5, out=out, delta=a), graph=True),
            t * width * (4 + 4 + 2 + 2))
 
     # the gated delta rule with one decay a head beside the one with a decay a key channel
@@ -785,18 +784,17 @@ def pegurax_kernel_table(size, device, peaks) -> Dict[str, dict]:
         for what, head in (("a decay a head", True), ("a decay a key channel; tanupel", False)):
             aa, bias = (a[:, :H].contiguous(), dt_bias[:H].contiguous()) if head else (a, dt_bias)
             bw(f"delta rule t={t}: recurrence, {what} ({n_seqs} sequences, {H} heads, state {d} x {dv})", timer.us(lambda: ops.delta_scan(
-                qkv, aa, b, bias, a_log, state, ctx, H, G, d, dv, head_decay=head), graph=few(t)),
+                qkv, aa, b, bias, a_log, state, ctx, H, G, d, dv, head_decay=head), graph=True),
                t * (channels * 4 + aa.shape[1] * 2 + H * dv * 4) + state_bytes)
             state.zero_()
         y = rand(t, H * dv, dtype=torch.float32)
         for act in ("silu", "sigmoid"):
             bw(f"delta rule t={t}: norm per head + {act} gate", timer.us(lambda: ops.head_norm_gate(y, z, norm_w, H, dv, 1e-5, ctx, act=act),
-                                                                     graph=few(t)), t * H * dv * (4 + 2 + 2))
+                                                                     graph=True), t * H * dv * (4 + 2 + 2))
 
-    # the selective scan beside Zeladra's state-space recurrence (as many state numbers, and at this width)
+    # the selective scan beside Zeladra's state-space recurrence (the last row of each: as many state numbers as that one's)
     scan = cfg["layers"][1]["mixer"]
-    N = scan["state"]
-    for inner in (scan["inner"], 2 * width):
+    for inner, N in ((scan["inner"], scan["state"]), (2 * width, scan["state"]), (2 * width, 128)):
         sstate = torch.zeros(DECODE_BATCH, inner * N + 3 * inner, dtype=torch.float32, device=device)
         vec = [rand(inner, dtype=torch.float32) for _ in range(2)]
         rates = -torch.exp(rand(inner, N, dtype=torch.float32))
@@ -804,11 +802,11 @@ def pegurax_kernel_table(size, device, peaks) -> Dict[str, dict]:
         for t, n_seqs in ((PREFILL_TOKENS, 1), (DECODE_BATCH, DECODE_BATCH)):
             ctx = context(t, n_seqs)
             proj, dt, low = rand(t, 2 * inner), rand(t, inner), rand(t, 2 * N)
-            bw(f"selective scan t={t}: convolution + SiLU ({inner} channels)", timer.us(lambda: ops.time_conv(
-                proj, 0, inner, cw, cb, sstate, inner * N, 4, ctx, act="silu", out_dtype=torch.bfloat16), graph=few(t)), t * inner * 4)
+            bw(f"selective scan t={t}: convolution + SiLU ({inner} channels, {N})", timer.us(lambda: ops.time_conv(
+                proj, 0, inner, cw, cb, sstate, inner * N, 4, ctx, act="silu", out_dtype=torch.bfloat16), graph=True), t * inner * 4)
             u = ops.time_conv(proj, 0, inner, cw, cb, sstate, inner * N, 4, ctx, act="silu", out_dtype=torch.bfloat16)
             bw(f"selective scan t={t}: recurrence and gate ({n_seqs} sequences, {inner} channels of {N})", timer.us(lambda: ops.selective_scan(
-                u, dt, low, 0, proj[:, inner:], vec[0], rates, vec[1], sstate, ctx, N), graph=few(t)),
+                u, dt, low, 0, proj[:, inner:], vec[0], rates, vec[1], sstate, ctx, N), graph=True),
                t * (inner * 8 + 4 * N) + n_seqs * inner * N * 8)
             sstate.zero_()
     ssm = zeladra_config(*size)["layers"][1]["mixer"]
@@ -822,14 +820,14 @@ def pegurax_kernel_table(size, device, peaks) -> Dict[str, dict]:
         proj = rand(t, cols)
         ctx = context(t, n_seqs)
         bw(f"state-space (zeladra) t={t}: convolution + SiLU ({sch} channels)", timer.us(lambda: ops.mamba2_conv(
-            proj, inner, sch, sconv_w, sconv_b, sstate, sH * sN * P, staps, ctx), graph=few(t)), t * sch * 6)
+            proj, inner, sch, sconv_w, sconv_b, sstate, sH * sN * P, staps, ctx), graph=True), t * sch * 6)
         xbc = ops.mamba2_conv(proj, inner, sch, sconv_w, sconv_b, sstate, sH * sN * P, staps, ctx)
 
         def recurrence():
             y = ops.mamba2_scan(xbc, proj, inner + sch, *vec, sstate, ctx, sH, sG, sN, P)
             return ops.gated_part_norm(y, proj[:, :inner], nw, 8, 1e-5, ctx)
         bw(f"state-space (zeladra) t={t}: recurrence, gate and norm ({n_seqs} sequences, {sH} heads, state {sN} x {P})",
-           timer.us(recurrence, graph=few(t)), t * (sch * 4 + inner * (4 + 4 + 2 + 2)) + n_seqs * sH * sN * P * 8)
+           timer.us(recurrence, graph=True), t * (sch * 4 + inner * (4 + 4 + 2 + 2)) + n_seqs * sH * sN * P * 8)
         sstate.zero_()
 
     # routed experts: weights on the inputs beside weights on the outputs
@@ -845,10 +843,10 @@ def pegurax_kernel_table(size, device, peaks) -> Dict[str, dict]:
         logits = ops.moe_logits(x, router)
         for score, weigh in (("sigmoid", True), ("softmax", False)):
             ids, weights = ops.moe_route(logits, None, top, ctx, score=score)
-            us = timer.us(lambda: ops.moe_experts(x, ids, weights, w1, w3, w2, w13, weigh_input=weigh), graph=few(t))
+            us = timer.us(lambda: ops.moe_experts(x, ids, weights, w1, w3, w2, w13, weigh_input=weigh), graph=True)
             touched = min(E, t * top)
             table[f"routed experts t={t}: {top} of {E} experts of {f} rows, weights on the {'inputs' if weigh else 'outputs; tanupel'}"] = dict(
-                choice_us=round(timer.us(lambda: ops.moe_route(logits, None, top, ctx, score=score), graph=few(t)), 1),
+                choice_us=round(timer.us(lambda: ops.moe_route(logits, None, top, ctx, score=score), graph=True), 1),
                 experts_us=round(us, 1), experts_tensor_frac=round(6 * t * top * f * width / (us * 1e-6) / tensor, 3),
                 experts_hbm_frac=round(touched * 3 * f * width * 2 / (us * 1e-6) / hbm, 3))
         for act in ("relu", "silu"):
@@ -858,7 +856,7 @@ def pegurax_kernel_table(size, device, peaks) -> Dict[str, dict]:
                     g = torch.empty(t, ffn, dtype=torch.bfloat16, device=device)
                     ops.silu_gate(ops.linear(x, wd13), g, 8, act=act)
                 return ops.linear(g, wd)
-            us = timer.us(dense, graph=few(t))
+            us = timer.us(dense, graph=True)
             table[f"dense gated feed-forward t={t}: {ffn} rows, {act}{' (llama)' if act == 'silu' else ''}"] = dict(
                 us=round(us, 1), tensor_frac=round(6 * t * ffn * width / (us * 1e-6) / tensor, 3),
                 hbm_frac=round(3 * ffn * width * 2 / (us * 1e-6) / hbm, 3))
