@@ -311,7 +311,8 @@ extern "C" int fg_attention_decode_bf16(const void* q, int q_stride, void* out, 
                                         softcap > 0.f ? scale / softcap : 0.f);
   FG_CHECK_LAUNCH("fg_attention_decode_bf16");
   dim3 cgrid(n_heads, n_seqs);
-  attention_combine_kernel<FG_HEAD_DIM><<<cgrid, COMBINE_THREADS, 0, stream>>>(
+  (window < 0 ? attention_combine_kernel<FG_HEAD_DIM, true>
+              : attention_combine_kernel<FG_HEAD_DIM, false>)<<<cgrid, COMBINE_THREADS, 0, stream>>>(
       scratch, (__nv_bfloat16*)out, out_stride, pos, seq_req, seq_tok, n_heads, window, max_splits, nullptr, status,
       out_freqs, keep_first, sinks);
   FG_CHECK_LAUNCH("fg_attention_combine");
@@ -364,8 +365,9 @@ extern "C" int fg_attention_decode_tma_bf16(const void* q, int q_stride, void* o
     FG_CHECK_ARG(scratch_floats >= fg_attention_decode_scratch_floats(n_seqs, max_splits, n_heads, max_pairs),
                  "fg_attention_decode_tma_bf16: scratch of %lld floats is too small", scratch_floats);
     const size_t psmem = decode_persistent_smem_bytes<FG_HEAD_DIM>(group);
-    auto pkern = attention_decode_persistent_kernel<FG_HEAD_DIM>;
-    static size_t pattr_set = 0;
+    auto pkern = window < 0 ? attention_decode_persistent_kernel<FG_HEAD_DIM, true> : attention_decode_persistent_kernel<FG_HEAD_DIM, false>;
+    static size_t pattr_sets[2] = {0, 0};
+    size_t& pattr_set = pattr_sets[window < 0];
     if (pattr_set < psmem) {
       cudaError_t e = cudaFuncSetAttribute(pkern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)psmem);
       FG_CHECK_ARG(e == cudaSuccess, "fg_attention_decode_tma_bf16: shared memory: %s", cudaGetErrorString(e));
@@ -395,7 +397,7 @@ extern "C" int fg_attention_decode_tma_bf16(const void* q, int q_stride, void* o
   }
   FG_CHECK_LAUNCH("fg_attention_decode_tma_bf16");
   dim3 cgrid(n_heads, n_seqs);
-  fg_launch_pdl(fg_mma::attention_combine_kernel<FG_HEAD_DIM>, cgrid, dim3(fg_mma::COMBINE_THREADS), 0, stream,
+  fg_launch_pdl(window < 0 ? fg_mma::attention_combine_kernel<FG_HEAD_DIM, true> : fg_mma::attention_combine_kernel<FG_HEAD_DIM, false>, cgrid, dim3(fg_mma::COMBINE_THREADS), 0, stream,
                 (const float*)partials, (__nv_bfloat16*)out, out_stride, pos, seq_req, seq_tok, n_heads, window,
                 max_splits, combine_pairs, status, out_freqs, 0, sinks);
   FG_CHECK_LAUNCH("fg_attention_combine");

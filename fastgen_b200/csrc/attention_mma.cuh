@@ -625,7 +625,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
 // request's own splits only, never on the batch.
 constexpr int COMBINE_THREADS = 256;
 
-template <int HD>
+template <int HD, bool CHUNKS>
 __global__ void __launch_bounds__(COMBINE_THREADS)
 attention_combine_kernel(const float* scratch, __nv_bfloat16* __restrict__ out, int out_stride,
                          const int* __restrict__ pos, const int* __restrict__ seq_req,
@@ -662,7 +662,7 @@ attention_combine_kernel(const float* scratch, __nv_bfloat16* __restrict__ out, 
   // a padding lane has no request: nothing is written for it (its token index may be any row,
   // also one that belongs to a request of the step)
   if (request < 0) return;
-  const int s_lo = first_visible(p, window) / DECODE_SPLIT;
+  const int s_lo = first_visible<CHUNKS>(p, window) / DECODE_SPLIT;
   int s_hi = p / DECODE_SPLIT;  // inclusive
   if (s_hi >= max_splits) {
     // the launch was sized for shorter requests: report instead of reading past the scratch

@@ -301,7 +301,7 @@ __device__ __forceinline__ uint32_t movmatrix_trans(uint32_t x) {
 template <int HD>
 constexpr int ps_blocks_per_sm() { return HD <= 64 ? 3 : 2; }
 
-template <int HD>
+template <int HD, bool CHUNKS>
 __global__ void __launch_bounds__(PS_THREADS, ps_blocks_per_sm<HD>())
 attention_decode_persistent_kernel(const __grid_constant__ CUtensorMap k_map,
                                    const __grid_constant__ CUtensorMap v_map, int layer,
@@ -342,7 +342,7 @@ attention_decode_persistent_kernel(const __grid_constant__ CUtensorMap k_map,
   // are the (request, split, kv head) triples that exist, numbered request by request, so
   // that block b takes items b, b + G, ... and every block gets the same number of them.
   // Positions are inputs of the step (no kernel of the step writes them).
-  auto first_split = [&](int p) { return first_visible(p, window) / SPLIT; };
+  auto first_split = [&](int p) { return first_visible<CHUNKS>(p, window) / SPLIT; };
   for (int sq = tid; sq < n_seqs; sq += PS_THREADS) s_pos[sq] = seq_req[sq] < 0 ? -1 : pos[seq_tok[sq]];
   __syncthreads();
   if (warp == 0) {
@@ -399,7 +399,7 @@ attention_decode_persistent_kernel(const __grid_constant__ CUtensorMap k_map,
     seq = lo;
     p = s_pos[seq];
     split = first_split(p) + (r - s_cum[seq]);
-    k_begin = first_visible(p, window);
+    k_begin = first_visible<CHUNKS>(p, window);
     return true;
   };
 

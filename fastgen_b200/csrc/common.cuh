@@ -126,9 +126,11 @@ __device__ __forceinline__ void store_from_f32(void* p, int dtype, size_t i, flo
 // The first position that an attention query at position p sees.  `window` > 0: the last `window` positions,
 // its own included; `window` < 0: those of its own chunk, chunks of -window positions counted from the
 // sequence's start; 0: all of them.  It never falls as p grows.
+// (CHUNKS false: the instantiation of a kernel for launches without chunks, which has no division in it.)
+template <bool CHUNKS = true>
 __device__ __forceinline__ int first_visible(int p, int window) {
   if (window > 0) return max(0, p - window + 1);
-  return window < 0 ? max(p, 0) / -window * -window : 0;
+  return CHUNKS && window < 0 ? max(p, 0) / -window * -window : 0;
 }
 
 __device__ __forceinline__ float warp_sum(float v) {
