@@ -12,7 +12,7 @@ Keys read: ``architecture``, ``vocab``, ``width``, ``norm.eps``, ``embedding.sca
   ``left{heads, kv_heads, dim, vdim, scale, rot{dims, base, scaling{factor, original, fast, slow}}, mask.size}``:
   grouped-query softmax attention inside chunks of ``mask.size`` positions, an RMS norm of queries and keys
   over their whole projection, a rotation of a head's first ``rot.dims`` dimensions (dimension ``i`` with
-  ``i + dims/2``, YaRN frequencies and magnitude), one added to the softmax's denominator;
+  ``i + dims/2``, YaRN frequencies and magnitude), a sink of score zero in every head's softmax;
   ``right{heads, kv_heads, dim, vdim, conv}``: the gated delta rule with one decay per head and a full
   SiLU gate (``parts/gated_delta.py``);
 * ``mamba1``: ``inner, state, dt_rank, conv``: the selective scan (``parts/selective_scan.py``);
